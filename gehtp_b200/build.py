@@ -19,6 +19,7 @@ UNITS = {
     "wt_parse.cpp": [],
     "executor.cu": [],
     "plan.cu": [],
+    "plan_rows.cu": [],
     "fuse.cu": [],
     "api_kernels.cu": [],
     "ops_elem.cu": ["--fmad=false"],
@@ -33,6 +34,11 @@ UNITS = {
     "ops_w4a16.cu": [],
     "w4a16_gemm_sm100.cu": [],
     "f16_gemm_sm100.cu": [],
+    "ops_rows.cu": [],
+    "linear_rows.cu": [],
+    "latent_attn.cu": [],
+    "latent_prefill.cu": [],
+    "channel_delta.cu": [],
     "tp.cu": [],
     "tp_p2p.cu": [],
 }
@@ -58,7 +64,8 @@ def _stale(src, obj):
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(verbose=False, force=False):
+def build(verbose=False, force=False, runner=True):
+    """Builds the library; runner=False leaves out the C++ host runner."""
     os.makedirs(OBJ, exist_ok=True)
     inc, lib = _nccl_dirs()
     nccl_flags = ["-I" + inc] if inc else []
@@ -91,6 +98,8 @@ def build(verbose=False, force=False):
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
     # host runner (job.txt / request-file protocols of the reference's device-side runners)
+    if not runner:
+        return OUT
     run_src = os.path.join(CSRC, "host", "gehtp_run.cpp")
     run_bin = os.path.join(os.path.dirname(OUT), "gehtp_run")
     if force or _stale(run_src, run_bin) or os.path.getmtime(OUT) > os.path.getmtime(run_bin):

@@ -4,6 +4,7 @@
 #include <stdint.h>
 #include <functional>
 #include <map>
+#include <memory>
 #include <string>
 #include <vector>
 #include "gehtp_cuda.h"
@@ -22,6 +23,7 @@ struct KvGeom {
 };
 
 struct W4Epilogue;
+struct RowsArgs;   // launchers_rows.h
 
 // One runlist op after planning: resolved device pointers baked into `launch`.
 struct PlanOp {
@@ -34,6 +36,11 @@ struct PlanOp {
     uint32_t out_bytes[2] = {0, 0};
     int kv_append_state = -1;   // AUTO append: host counter check / bump
     int kv_gather_state = -1;   // AUTO gather: host counter check
+    // row-count runlists: bytes of the outputs per row (out_bytes is then the largest size), and which count they follow
+    uint32_t out_row_bytes[2] = {0, 0}, out_rows_arg[2] = {0, 0};
+    int pos_append_state = -1;  // appends the run's rows at the state's counter: host check for room
+    uint32_t adv_first = 0, adv_n = 0, adv_rows = 0;   // OP_STATE_ADVANCE: host mirror of the counters
+    std::shared_ptr<RowsArgs> rows_args;               // resolved operands of a row-count op, for fusion
     uint32_t w4_m = 0;          // M of a W4A16 matmul (reported through engine_m)
     // a W4A16 matmul at GEMM row counts: the tcgen05 GEMM with an epilogue of the caller's (false: shape not taken)
     // `a_src` / `a_d` != 0: read the activations from a_src, stored [K / a_d][M][a_d], instead of the op's own operand
@@ -112,12 +119,18 @@ struct Engine {
     const uint8_t* ext_in_dev = nullptr;
     const uint8_t* ext_wgt = nullptr;
 
-    // CUDA graph of a whole run
-    cudaGraphExec_t graph = nullptr;
-    uint32_t graph_out_temp = kNoOff;
-    bool graph_has_in = false, graph_has_out = false;
-    uint32_t warm_runs = 0;
-    unsigned long long graph_launches = 0;  // kernels inside the captured graph
+    // row-count runlists: limits of the blob (0: an ordinary blob) and the counts of the next run
+    uint32_t max_rows = 0, max_sel = 0, run_rows = 0, run_sel = 0;
+
+    // CUDA graphs of whole runs, one per I/O binding and row count
+    struct RunGraph {
+        cudaGraphExec_t exec;
+        uint32_t out_temp, rows, sel;
+        bool has_in, has_out;
+        unsigned long long launches;         // kernels inside the captured graph
+    };
+    std::vector<RunGraph> graphs;
+    std::map<uint64_t, uint32_t> warm_runs;  // whole eager runs per (rows, sel)
 
     // per-unit CUDA event profiling (gehtp_cuda_run_profiled)
     struct ProfEvent { uint32_t op; cudaEvent_t e0, e1; };
@@ -150,6 +163,7 @@ int read_status(char* err, size_t errn);   // after a stream sync: 0, or the fai
 // plan.cu
 int build_plan(const wt_blob* b, char* err, size_t errn);
 void drop_plan(bool keep_states);
+void drop_graphs();
 // tp.cu
 extern std::vector<uint8_t> g_allreduce_after;   // per op: 1 = all-reduce its first output over the ranks
 // Fewest rows for which a W4A16 matmul goes to the tcgen05 GEMM (TMA zero-fills the rows a 128-row tile has
@@ -168,6 +182,11 @@ bool tp_p2p_allreduce_f16(cudaStream_t st, void* buf, size_t elems);
 void tp_p2p_shutdown();
 bool tp_p2p_add_rmsnorm(cudaStream_t st, const uint16_t* a, uint16_t* r, const uint16_t* g, const uint16_t* b,
                         uint16_t* sum_out, uint16_t* y, uint32_t rows, uint32_t width);
+// Most rows for which a whole run of a row-count runlist is captured: attention over more rows picks its launches by
+// the host's position count, which a replay would not follow.
+constexpr uint32_t kGraphRows = 8;
+// the value of a row argument in the coming run
+inline uint32_t rows_of(uint32_t arg) { return arg == WT_ROWS_AUTO ? g.run_rows : arg == WT_SEL_AUTO ? g.run_sel : arg; }
 // fuse.cu
 void fuse_analyze(const wt_blob* b, const std::vector<PlanOp>& meas, std::vector<uint8_t>& internal, std::vector<uint8_t>& dead);
 void fuse_materialize(const wt_blob* b);

@@ -176,14 +176,40 @@ static int host_precheck(const PlanOp& p, char* err, size_t errn) {
             return -1;
         }
     }
+    if (p.pos_append_state >= 0) {
+        uint32_t si = (uint32_t)p.pos_append_state, n = rows_of(WT_ROWS_AUTO);
+        if (g.st_count[si] + n > g.kv[si].nslots) {
+            std::snprintf(m, sizeof m, "append of %u rows to state %u count=%u nslots=%u (context too long)", n, si, g.st_count[si], g.kv[si].nslots);
+            set_err(err, errn, m);
+            return -1;
+        }
+    }
     return 0;
+}
+
+// Host mirror of OP_STATE_ADVANCE, in step with the launch that advances the device counters.
+static void host_advance(const PlanOp& p, int sign) {
+    for (uint32_t k = 0; k < p.adv_n; k++) g.st_count[p.adv_first + k] += sign * rows_of(p.adv_rows);
+}
+
+// Undoes the counter bookkeeping of a capture whose graph never ran.
+static void undo_counters(const wt_blob* b) {
+    for (uint32_t i = 0; i < b->n_ops; i++) {
+        if (g.plan[i].kv_append_state >= 0) g.st_count[g.plan[i].kv_append_state]--;
+        host_advance(g.plan[i], -1);
+    }
+}
+
+void drop_graphs() {
+    for (auto& gr : g.graphs) cudaGraphExecDestroy(gr.exec);
+    g.graphs.clear();
 }
 
 static void note_outputs(const PlanOp& p) {
     for (int k = 0; k < 2; k++) {
         uint32_t id = p.out_id[k];
         if (id == kNoOff) continue;
-        g.temp_last[id] = p.out_bytes[k];
+        g.temp_last[id] = p.out_row_bytes[k] ? p.out_row_bytes[k] * rows_of(p.out_rows_arg[k]) : p.out_bytes[k];
         if (g.temp_cap[id] < p.out_bytes[k]) g.temp_cap[id] = p.out_bytes[k];
     }
 }
@@ -239,6 +265,7 @@ static int queue_range(uint32_t first, uint32_t count, bool fuse, bool per_op_sy
                 }
             }
             if (ev1) cudaEventRecord(ev1, g.stream);
+            if (!rc) for (PlanOp* q : pending) host_advance(*q, 1);
             pending.clear();
         }
 
@@ -346,18 +373,20 @@ static int run_impl(const wt_blob* b, uint32_t first, uint32_t count, const void
     const bool timing = op_us || g.ts_buf;
     const bool whole = first == 0 && count == b->n_ops;
     const bool has_in = in_host || in_dev;
-    const bool eager_only = timing || hooks_active() || g.trace_on || !g.opt_graph || !whole || g.prof_ms;
+    const uint32_t rows = g.run_rows, sel = g.run_sel;
+    const bool eager_only = timing || hooks_active() || g.trace_on || !g.opt_graph || !whole || g.prof_ms || rows > kGraphRows;
 
     int rc = 0;
     // Device-side input and output copies stay outside the graph (their pointers
     // may change from run to run); host staging goes through fixed pinned buffers
     // and is part of it.
-    if (!eager_only && g.graph && (g.graph_out_temp != out_temp || g.graph_has_in != (in_host != nullptr) ||
-                                   g.graph_has_out != (out_host != nullptr))) {
-        cudaGraphExecDestroy(g.graph);   // same blob, different I/O binding: capture again
-        g.graph = nullptr;
-    }
-    if (!eager_only && g.graph) {
+    // Another I/O binding or row count of the same blob has a graph of its own.
+    Engine::RunGraph* have = nullptr;
+    if (!eager_only)
+        for (auto& gr : g.graphs)
+            if (gr.out_temp == out_temp && gr.rows == rows && gr.sel == sel && gr.has_in == (in_host != nullptr) &&
+                gr.has_out == (out_host != nullptr)) have = &gr;
+    if (have) {
         // replay: host bookkeeping first, then one launch
         for (uint32_t i = 0; i < b->n_ops; i++) {
             PlanOp& q = g.plan[i];
@@ -367,14 +396,15 @@ static int run_impl(const wt_blob* b, uint32_t first, uint32_t count, const void
             bump_stat(q.stat);
             g.st.ops++;
             note_outputs(q);
+            host_advance(q, 1);
         }
         if (in_host) {
             for (auto& kv : g.d_ext)
                 if (b->slots[kv.first].addr == WT_SLOT_EXT_IN) std::memcpy(g.h_in, in_host, b->slots[kv.first].len);
         }
         if (in_dev) stage_inputs(b, nullptr, in_dev);
-        cudaGraphLaunch(g.graph, g.stream);
-        g_launches += g.graph_launches;
+        cudaGraphLaunch(have->exec, g.stream);
+        g_launches += have->launches;
         if (out_dev && out_temp < kMaxTemps && g.temp_cap[out_temp])
             cudaMemcpyAsync(out_dev, g.temp_dev[out_temp], g.temp_last[out_temp], cudaMemcpyDeviceToDevice, g.stream);
         if (!sync_end) return 0;
@@ -384,7 +414,8 @@ static int run_impl(const wt_blob* b, uint32_t first, uint32_t count, const void
     }
 
     // a run that could be graphed later is captured on its second eager pass
-    const bool capture = !eager_only && !g.graph && g.warm_runs >= 1;
+    const uint64_t warm_key = (uint64_t)rows << 32 | sel;
+    const bool capture = !eager_only && g.warm_runs[warm_key] >= 1;
     uint32_t out_bytes_planned = 0;
     if (capture) {
         if (in_host)
@@ -448,22 +479,20 @@ static int run_impl(const wt_blob* b, uint32_t first, uint32_t count, const void
             cudaGetLastError();
             g.opt_graph = 0;  // this blob cannot be graphed; stay eager
             if (rc != 0) return rc;
-            // host counters were advanced while capturing: undo, then run eagerly
-            for (uint32_t i = 0; i < b->n_ops; i++)
-                if (g.plan[i].kv_append_state >= 0) g.st_count[g.plan[i].kv_append_state]--;
+            undo_counters(b);   // advanced while capturing; now run eagerly
             return run_impl(b, first, count, in_host, in_dev, out_host, out_dev, out_temp, sync_end, engine_m, op_us, err, errn);
         }
-        ce = cudaGraphInstantiate(&g.graph, graph, 0);
+        cudaGraphExec_t exec = nullptr;
+        ce = cudaGraphInstantiate(&exec, graph, 0);
         cudaGraphDestroy(graph);
         if (ce != cudaSuccess) {
-            g.graph = nullptr; g.opt_graph = 0; cudaGetLastError();
-            for (uint32_t i = 0; i < b->n_ops; i++)
-                if (g.plan[i].kv_append_state >= 0) g.st_count[g.plan[i].kv_append_state]--;
+            g.opt_graph = 0; cudaGetLastError();
+            undo_counters(b);
             return run_impl(b, first, count, in_host, in_dev, out_host, out_dev, out_temp, sync_end, engine_m, op_us, err, errn);
         }
-        g.graph_launches = g_launches - launches0;
-        g.graph_out_temp = out_temp; g.graph_has_in = in_host != nullptr; g.graph_has_out = out_host != nullptr;
-        cudaGraphLaunch(g.graph, g.stream);
+        if (g.graphs.size() >= 16) { cudaGraphExecDestroy(g.graphs.front().exec); g.graphs.erase(g.graphs.begin()); }
+        g.graphs.push_back({exec, out_temp, rows, sel, in_host != nullptr, out_host != nullptr, g_launches - launches0});
+        cudaGraphLaunch(exec, g.stream);
         if (out_dev && out_temp < kMaxTemps && g.temp_cap[out_temp])
             cudaMemcpyAsync(out_dev, g.temp_dev[out_temp], g.temp_last[out_temp], cudaMemcpyDeviceToDevice, g.stream);
         if (!sync_end) return 0;
@@ -472,7 +501,7 @@ static int run_impl(const wt_blob* b, uint32_t first, uint32_t count, const void
         return rc;
     }
     if (rc != 0) { cudaStreamSynchronize(g.stream); return rc; }
-    if (whole) g.warm_runs++;
+    if (whole) g.warm_runs[warm_key]++;
     if (out_dev && out_temp < kMaxTemps && g.temp_cap[out_temp])
         cudaMemcpyAsync(out_dev, g.temp_dev[out_temp], g.temp_last[out_temp], cudaMemcpyDeviceToDevice, g.stream);
     if (out_host && out_temp < kMaxTemps && g.temp_cap[out_temp]) {
@@ -553,7 +582,7 @@ void wt_exec_state_reset(void) {
     for (uint32_t i = 0; i < g.n_states; i++) {
         cudaMemsetAsync(g.st_buf[i], 0, g.st_bytes[i], g.stream);
         g.st_count[i] = 0;
-        if (g.kv[i].ready) cudaMemsetAsync(g.kv[i].posmap, 0xFF, (size_t)g.kv[i].nslots * 4, g.stream);
+        if (g.kv[i].ready && g.kv[i].posmap) cudaMemsetAsync(g.kv[i].posmap, 0xFF, (size_t)g.kv[i].nslots * 4, g.stream);
     }
     cudaMemsetAsync(g.d_st_count, 0, 2 * WT_MAX_STATES * sizeof(uint32_t), g.stream);
     cudaStreamSynchronize(g.stream);
@@ -616,7 +645,21 @@ void gehtp_cuda_set_fusion(int on) {
 }
 void gehtp_cuda_set_graph(int on) {
     g.opt_graph = on ? 1 : 0;
-    if (!on && g.graph) { cudaGraphExecDestroy(g.graph); g.graph = nullptr; }
+    if (!on) drop_graphs();
+}
+int gehtp_cuda_set_rows(const struct wt_blob* b, uint32_t rows, uint32_t sel, char* err, size_t errn) {
+    if (!b) { set_err(err, errn, "null blob"); return -1; }
+    if (!ensure_device(err, errn) || ensure_plan(b, err, errn) != 0) return -1;
+    if (!g.max_rows) { set_err(err, errn, "not a row-count runlist"); return -1; }
+    if (!rows || rows > g.max_rows || sel > g.max_sel || sel > rows) {
+        char m[128];
+        std::snprintf(m, sizeof m, "rows %u of %u, picked %u of %u", rows, g.max_rows, sel, g.max_sel);
+        set_err(err, errn, m);
+        return -1;
+    }
+    g.run_rows = rows;
+    g.run_sel = sel;
+    return 0;
 }
 uint64_t gehtp_cuda_launch_count(void) { return g_launches; }
 uint32_t gehtp_cuda_fused_ops(void) { return g.fused_ops; }

@@ -25,7 +25,8 @@
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include "common.cuh"
-#include "launchers.h"
+#include "launchers_rows.h"
+#include "rows_common.cuh"
 #include "sm100_umma.cuh"
 #include "w4_stream.cuh"
 
@@ -53,11 +54,67 @@ struct __align__(8) FBarriers {
 
 __device__ __forceinline__ uint32_t pack2(float a, float b) { return (uint32_t)f2h(a) | ((uint32_t)f2h(b) << 16); }
 
+// Operand and output types of the kernel. EDGE: N need not be a multiple of the tile width nor K of 64 (the tensor
+// maps zero-fill what lies outside), the epilogue checks its columns; store8 writes 8 neighbouring outputs.
+struct IoF16 {                                    // the runlist's fp16 matmul
+    typedef uint16_t Out;
+    static constexpr bool EDGE = false;
+    static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
+    static constexpr uint32_t IDESC = 0;
+    static __device__ __forceinline__ void store8(Out* p, const float* v, uint32_t) {
+        *(uint4*)p = make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7]));
+    }
+    static __device__ __forceinline__ void store4(Out* p, const float* v, uint32_t) { *(uint2*)p = make_uint2(pack2(v[0], v[1]), pack2(v[2], v[3])); }
+};
+template <bool RELU2>
+__device__ __forceinline__ float lin_act(float v) {
+    if (!RELU2) return v;
+    v = fmaxf(v, 0.0f);
+    return v * v;
+}
+constexpr uint32_t IDESC_BF16 = (1u << 7) | (1u << 10);      // A and B are bf16
+template <bool RELU2>
+struct IoBf16 {                                   // bf16 in, bf16 out
+    typedef uint16_t Out;
+    static constexpr bool EDGE = true;
+    static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    static constexpr uint32_t IDESC = IDESC_BF16;
+    static __device__ __forceinline__ uint32_t pk(float a, float b) { return pack_bf2(lin_act<RELU2>(a), lin_act<RELU2>(b)); }
+    static __device__ __forceinline__ void store8(Out* p, const float* v, uint32_t left) {
+        if (left >= 8 && ((uintptr_t)p & 15u) == 0) { *(uint4*)p = make_uint4(pk(v[0], v[1]), pk(v[2], v[3]), pk(v[4], v[5]), pk(v[6], v[7])); return; }
+#pragma unroll
+        for (uint32_t i = 0; i < 8; i++) if (i < left) p[i] = f2bf(lin_act<RELU2>(v[i]));
+    }
+    static __device__ __forceinline__ void store4(Out* p, const float* v, uint32_t left) {
+#pragma unroll
+        for (uint32_t i = 0; i < 4; i++) if (i < left) p[i] = f2bf(lin_act<RELU2>(v[i]));
+    }
+};
+template <bool RELU2>
+struct IoBf16F32 {                                // bf16 in, fp32 out
+    typedef float Out;
+    static constexpr bool EDGE = true;
+    static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    static constexpr uint32_t IDESC = IDESC_BF16;
+    static __device__ __forceinline__ void store4(Out* p, const float* v, uint32_t left) {
+        if (left >= 4 && ((uintptr_t)p & 15u) == 0) {
+            *(float4*)p = make_float4(lin_act<RELU2>(v[0]), lin_act<RELU2>(v[1]), lin_act<RELU2>(v[2]), lin_act<RELU2>(v[3]));
+            return;
+        }
+#pragma unroll
+        for (uint32_t i = 0; i < 4; i++) if (i < left) p[i] = lin_act<RELU2>(v[i]);
+    }
+    static __device__ __forceinline__ void store8(Out* p, const float* v, uint32_t left) {
+        store4(p, v, left);
+        if (left > 4) store4(p + 4, v + 4, left - 4);
+    }
+};
+
 // y rows are ldy elements apart (the SPLIT form writes N columns of a row of N_full).
-template <int MH, int BN>
+template <int MH, int BN, class IO>
 __global__ void __launch_bounds__(NTHREADS, 1)
 f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_w,
-                      uint16_t* __restrict__ y, uint32_t M, uint32_t K, uint32_t N, uint32_t ldy, unsigned int* status,
+                      typename IO::Out* __restrict__ y, uint32_t M, uint32_t K, uint32_t N, uint32_t ldy, unsigned int* status,
                       uint32_t S, float* __restrict__ part) {
     using C = FCfg<MH, BN>;
     constexpr int STAGES = C::STAGES, NBUF = C::NBUF, A_BYTES = C::A_BYTES, B_BYTES = C::B_BYTES;
@@ -70,8 +127,8 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
     volatile uint32_t* abort_flag = &bars->abort_flag;
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t KG = K / BK;
-    const uint32_t m_tiles = (M + 128 * MH - 1) / (128 * MH), tiles = m_tiles * (N / BN);
+    const uint32_t KG = IO::EDGE ? (K + BK - 1) / BK : K / BK;
+    const uint32_t m_tiles = (M + 128 * MH - 1) / (128 * MH), tiles = m_tiles * (IO::EDGE ? (N + BN - 1) / BN : N / BN);
     // Split K (S > 1): a work item is (tile, run of K/64/S k blocks), item = run * tiles + tile; a run leaves its fp32
     // partial sums in part[run][row][N] and f16_splitk_reduce_kernel adds the runs in order.
     const uint32_t items = tiles * S, KGS = KG / S;
@@ -132,7 +189,7 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
                     for (uint32_t k4 = 0; k4 < BK / 16; k4++) {
 #pragma unroll
                         for (int h = 0; h < MH; h++)
-                            umma_f16(acc + h * BN, da0 + (uint64_t)(h * (HALF_A_BYTES >> 4) + k4 * 2), db0 + (uint64_t)(k4 * 2), idesc_f16(BN),
+                            umma_f16(acc + h * BN, da0 + (uint64_t)(h * (HALF_A_BYTES >> 4) + k4 * 2), db0 + (uint64_t)(k4 * 2), idesc_f16(BN) | IO::IDESC,
                                      (kb | k4) ? 1u : 0u);
                     }
                     umma_commit(&bars->empty[s]);
@@ -172,18 +229,22 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
                           "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
                         : "r"(taddr));
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    const uint32_t n = n0 + c * 32;
                     if (m < M && S > 1) {
-                        uint4* dst = (uint4*)(part + ((size_t)run * M + m) * N + n0 + c * 32);
+                        // rows of the partial sums are N rounded up to 4 floats apart
+                        const uint32_t np = IO::EDGE ? (N + 3) & ~3u : N;
+                        uint4* dst = (uint4*)(part + ((size_t)run * M + m) * np + n);
 #pragma unroll
-                        for (int q = 0; q < 8; q++) dst[q] = make_uint4(v[4 * q], v[4 * q + 1], v[4 * q + 2], v[4 * q + 3]);
+                        for (int q = 0; q < 8; q++)
+                            if (!IO::EDGE || n + 4 * q < np) dst[q] = make_uint4(v[4 * q], v[4 * q + 1], v[4 * q + 2], v[4 * q + 3]);
                     } else if (m < M) {
-                        uint4* dst = (uint4*)(y + (size_t)m * ldy + n0 + c * 32);     // 16-byte aligned: y is, ldy is a multiple of 8
+                        typename IO::Out* dst = y + (size_t)m * ldy + n;     // fp16: 16-byte aligned, y is and ldy is a multiple of 8
+                        float f[32];
+#pragma unroll
+                        for (int q = 0; q < 32; q++) f[q] = __uint_as_float(v[q]);
 #pragma unroll
                         for (int q = 0; q < 4; q++)
-                            dst[q] = make_uint4(pack2(__uint_as_float(v[8 * q]), __uint_as_float(v[8 * q + 1])),
-                                                pack2(__uint_as_float(v[8 * q + 2]), __uint_as_float(v[8 * q + 3])),
-                                                pack2(__uint_as_float(v[8 * q + 4]), __uint_as_float(v[8 * q + 5])),
-                                                pack2(__uint_as_float(v[8 * q + 6]), __uint_as_float(v[8 * q + 7])));
+                            if (!IO::EDGE || n + 8 * q < N) IO::store8(dst + 8 * q, f + 8 * q, IO::EDGE ? N - n - 8 * q : 8);
                     }
                 }
             }
@@ -200,32 +261,35 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
     }
 }
 
-bool make_map(CUtensorMap* tm, const uint16_t* base, uint32_t rows, uint32_t K, uint32_t box_rows) {
+bool make_map(CUtensorMap* tm, CUtensorMapDataType type, const uint16_t* base, uint32_t rows, uint32_t K, uint32_t ld, uint32_t box_rows) {
     EncodeTiledFn enc = encode_fn();
     if (!enc) return false;
     cuuint64_t dims[2] = {K, rows};
-    cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+    cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
     cuuint32_t box[2] = {BK, box_rows};
     cuuint32_t estr[2] = {1, 1};
-    return enc(tm, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void*)base, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    return enc(tm, type, 2, (void*)base, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-// y[m][n] (rows ldy apart) = sum over the runs of part[run][m][n], in run order
+// y[m][n] (rows ldy apart) = sum over the runs of part[run][m][n], in run order; 4 columns per thread
+template <class IO>
 __global__ void __launch_bounds__(256)
-f16_splitk_reduce_kernel(const float* __restrict__ part, uint16_t* __restrict__ y, uint32_t M, uint32_t N, uint32_t ldy, uint32_t S) {
+f16_splitk_reduce_kernel(const float* __restrict__ part, typename IO::Out* __restrict__ y, uint32_t M, uint32_t N, uint32_t ldy, uint32_t S) {
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     asm volatile("griddepcontrol.wait;" ::: "memory");
-    const size_t quads = (size_t)M * N / 4, plane = quads;
-    const uint32_t nq = N / 4;
+    const uint32_t nq = (N + 3) / 4;
+    const size_t quads = (size_t)M * nq, plane = quads;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < quads; i += (size_t)gridDim.x * blockDim.x) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
         for (uint32_t r = 0; r < S; r++) {
             const float4 p = __ldcg((const float4*)part + r * plane + i);
             acc.x += p.x; acc.y += p.y; acc.z += p.z; acc.w += p.w;
         }
-        const size_t m = i / nq, n = (i % nq) * 4;
-        *(uint2*)(y + m * ldy + n) = make_uint2(pack2(acc.x, acc.y), pack2(acc.z, acc.w));
+        const size_t m = i / nq;
+        const uint32_t n = (uint32_t)(i % nq) * 4;
+        const float v[4] = {acc.x, acc.y, acc.z, acc.w};
+        IO::store4(y + m * ldy + n, v, N - n);
     }
 }
 
@@ -248,23 +312,24 @@ SplitScratch* split_scratch(cudaStream_t st, size_t need) {
     return &sc;
 }
 
-template <int MH, int BN>
-bool launch(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint16_t* y, uint32_t M, uint32_t K, uint32_t N, uint32_t ldy,
+template <int MH, int BN, class IO>
+bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w, typename IO::Out* y, uint32_t M, uint32_t K, uint32_t N, uint32_t ldy,
             unsigned int* status, int sms) {
     using C = FCfg<MH, BN>;
     CUtensorMap ta, tw;
-    if (!make_map(&ta, a, M, K, 128) || !make_map(&tw, w, N, K, BN)) return false;
+    if (!make_map(&ta, IO::MAP, a, M, K, lda, 128) || !make_map(&tw, IO::MAP, w, N, K, K, BN)) return false;
     const size_t smem = 1024 + (size_t)C::STAGES * (C::A_BYTES + C::B_BYTES) + sizeof(FBarriers) + 16;
     static int have[64] = {};
-    if (!ensure_dyn_smem(f16_gemm_sm100_kernel<MH, BN>, smem, have)) return false;
-    const uint32_t tiles = ((M + 128 * MH - 1) / (128 * MH)) * (N / BN), KG = K / BK;
+    if (!ensure_dyn_smem(f16_gemm_sm100_kernel<MH, BN, IO>, smem, have)) return false;
+    const uint32_t tiles = ((M + 128 * MH - 1) / (128 * MH)) * ((N + BN - 1) / BN), KG = (K + BK - 1) / BK;
+    const uint32_t np = (N + 3) & ~3u;
     // Split K while the tiles alone leave SMs idle (same rule as the W4A16 GEMM): the divisor of K/64 that makes
     // (items per CTA) x (k blocks per item + set-up) smallest, a run at least one trip round the ring, partial sums <= 64 MB.
     uint32_t S = 1;
     if (tiles < (uint32_t)sms) {
         float best = (float)(KG + 4);
         for (uint32_t c = 2; c <= 32 && c <= KG; c++) {
-            if (KG % c || KG / c < (uint32_t)C::STAGES || (size_t)c * M * N * sizeof(float) > ((size_t)64 << 20)) continue;
+            if (KG % c || KG / c < (uint32_t)C::STAGES || (size_t)c * M * np * sizeof(float) > ((size_t)64 << 20)) continue;
             const uint32_t rounds = (tiles * c + sms - 1) / sms;
             const float cost = (float)rounds * (float)(KG / c + 4) + 0.75f * (float)c + 6.0f;
             if (cost < best) { best = cost; S = c; }
@@ -272,21 +337,21 @@ bool launch(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint16_t* y, 
     }
     float* part = nullptr;
     if (S > 1) {
-        SplitScratch* ss = split_scratch(st, (size_t)S * M * N * sizeof(float));
+        SplitScratch* ss = split_scratch(st, (size_t)S * M * np * sizeof(float));
         if (ss) part = ss->part; else S = 1;
     }
     const uint32_t items = tiles * S;
     const uint32_t grid = items < (uint32_t)sms ? items : (uint32_t)sms;
-    if (launch_pdl(f16_gemm_sm100_kernel<MH, BN>, dim3(grid), dim3(NTHREADS), smem, st, ta, tw, y, M, K, N, ldy, status, S, part) != cudaSuccess) {
+    if (launch_pdl(f16_gemm_sm100_kernel<MH, BN, IO>, dim3(grid), dim3(NTHREADS), smem, st, ta, tw, y, M, K, N, ldy, status, S, part) != cudaSuccess) {
         cudaGetLastError();
         return false;
     }
     g_launches++;
     if (S > 1) {
-        const size_t quads = (size_t)M * N / 4;
+        const size_t quads = (size_t)M * np / 4;
         uint32_t rg = (uint32_t)((quads + 255) / 256);
         if (rg > (uint32_t)sms * 8) rg = (uint32_t)sms * 8;
-        if (launch_pdl(f16_splitk_reduce_kernel, dim3(rg), dim3(256), 0, st, (const float*)part, y, M, N, ldy, S) != cudaSuccess) {
+        if (launch_pdl(f16_splitk_reduce_kernel<IO>, dim3(rg), dim3(256), 0, st, (const float*)part, y, M, N, ldy, S) != cudaSuccess) {
             cudaGetLastError();
             return false;
         }
@@ -424,6 +489,24 @@ bool launch_gemv(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint16_t
     return true;
 }
 
+// tile shape by the number of tiles it gives
+template <class IO>
+bool launch_tiles(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w, typename IO::Out* y, uint32_t M, uint32_t K, uint32_t N,
+                  uint32_t ldy, unsigned int* status) {
+    static int sms_of[64] = {};
+    int dev = 0;
+    cudaGetDevice(&dev);
+    int& sms = sms_of[dev & 63];
+    if (!sms) {
+        cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+        if (sms <= 0) sms = 148;
+    }
+    const uint32_t t256 = ((M + 255) / 256) * ((N + 255) / 256), t128 = ((M + 255) / 256) * ((N + 127) / 128);
+    if ((IO::EDGE || N % 256 == 0) && M > 128 && t256 >= (uint32_t)sms) return launch<2, 256, IO>(st, a, lda, w, y, M, K, N, ldy, status, sms);
+    if (M > 128 && t128 >= (uint32_t)sms) return launch<2, 128, IO>(st, a, lda, w, y, M, K, N, ldy, status, sms);
+    return launch<1, 128, IO>(st, a, lda, w, y, M, K, N, ldy, status, sms);
+}
+
 }  // namespace
 
 // Y[M, N] (rows ldy apart) = A[M, K] . W^T, W stored [N, K]. false: shape or alignment outside what the
@@ -437,18 +520,19 @@ bool k_matmul_f16_nk(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint
         return M <= 4 ? launch_gemv<4>(st, a, w, y, M, K, N, ldy) : launch_gemv<8>(st, a, w, y, M, K, N, ldy);
     }
     if (M < 128 || K % BK || N % 128 || (ldy & 7u) || ((uintptr_t)y & 15u)) return false;
-    static int sms_of[64] = {};
-    int dev = 0;
-    cudaGetDevice(&dev);
-    int& sms = sms_of[dev & 63];
-    if (!sms) {
-        cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-        if (sms <= 0) sms = 148;
-    }
-    const uint32_t t256 = ((M + 255) / 256) * (N / 256), t128 = ((M + 255) / 256) * (N / 128);
-    if (N % 256 == 0 && M > 128 && t256 >= (uint32_t)sms) return launch<2, 256>(st, a, w, y, M, K, N, ldy, status, sms);
-    if (M > 128 && t128 >= (uint32_t)sms) return launch<2, 128>(st, a, w, y, M, K, N, ldy, status, sms);
-    return launch<1, 128>(st, a, w, y, M, K, N, ldy, status, sms);
+    return launch_tiles<IoF16>(st, a, K, w, y, M, K, N, ldy, status);
+}
+
+// The same kernel on bf16 operands with the outputs of a row-count projection: any N, K a multiple of 8 (16-byte rows),
+// any row count (a tile's missing rows are zero-filled).
+bool k_linear_sm100(cudaStream_t st, const LinearArgs& a, uint32_t M, unsigned int* status) {
+    if (!a.x_bf16 || !M || (a.K & 7u) || (a.xs & 7u) || ((((uintptr_t)a.x) | ((uintptr_t)a.w)) & 15u)) return false;
+    const uint16_t* x = (const uint16_t*)a.x;
+    if (a.y_bf16)
+        return a.relu2 ? launch_tiles<IoBf16<true>>(st, x, a.xs, a.w, (uint16_t*)a.y, M, a.K, a.N, a.ys, status)
+                       : launch_tiles<IoBf16<false>>(st, x, a.xs, a.w, (uint16_t*)a.y, M, a.K, a.N, a.ys, status);
+    return a.relu2 ? launch_tiles<IoBf16F32<true>>(st, x, a.xs, a.w, (float*)a.y, M, a.K, a.N, a.ys, status)
+                   : launch_tiles<IoBf16F32<false>>(st, x, a.xs, a.w, (float*)a.y, M, a.K, a.N, a.ys, status);
 }
 
 }  // namespace gehtp

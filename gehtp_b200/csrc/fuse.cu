@@ -17,6 +17,8 @@
 //   prefill q|k|v head  SPLIT x3 + two rotary chains (17 ops) -> one kernel
 //   transposition + GEMM  [heads][rows][d] -> [rows][heads d] in front of a W4A16 GEMM -> the GEMM reads the
 //                       untransposed tensor through a three-dimensional tensor map
+//   latent attention    LATENT_APPEND + LATENT_ATTEND of a row-count runlist -> for few rows: append and query absorption
+//                       in one kernel, split attention over the cached rows, merge with the value up-projection
 // and marks the data-movement ops whose result is a constant of the blob (fold_constants).
 //
 // A chain is fused only when every intermediate temp is consumed inside the
@@ -29,6 +31,7 @@
 #include <utility>
 #include "engine.h"
 #include "launchers_attn.h"
+#include "launchers_rows.h"
 #include "launchers_w4.h"
 
 namespace gehtp {
@@ -134,7 +137,8 @@ struct Span {
     int kind;                // 0 decode attention, 1 swiglu, 2 add+norm, 3 rotary, 4 prefill attention,
                              // 5 prefill split + rotary of q|k|v, 6 swiglu tail behind two GEMMs,
                              // 7 [head][row][d] -> [row][head * d] transposition in front of a W4A16 GEMM,
-                             // 8 per-row SLICE + ARGMAX of a matrix joined by a CONCAT tree (greedy sampling of a batch)
+                             // 8 per-row SLICE + ARGMAX of a matrix joined by a CONCAT tree (greedy sampling of a batch),
+                             // 9 latent append + attention of a row-count runlist
     uint32_t first, count;
     std::vector<uint32_t> ops;
     // attention
@@ -517,6 +521,20 @@ bool match_add_norm(const Graph& G, uint32_t i, Span& sp) {
     return true;
 }
 
+// LATENT_APPEND directly in front of the LATENT_ATTEND of its state and queries
+bool match_latent_step(const Graph& G, uint32_t i, Span& sp) {
+    const wt_blob* b = G.b;
+    if (i + 1 >= b->n_ops) return false;
+    const wt_op &ap = b->ops[i], &at = b->ops[i + 1];
+    if (ap.opcode != OP_LATENT_APPEND || at.opcode != OP_LATENT_ATTEND) return false;
+    if (at.args[0] != ap.args[3] || at.args[1] != ap.args[4] || at.args[2] != ap.args[5]) return false;
+    for (int k = 6; k < 10; k++) if (ap.args[k] != at.args[k]) return false;      // rows, heads, dim, rot
+    if (ap.args[10] != at.args[11] || ap.args[12] != at.args[13]) return false;   // rank, type
+    sp.kind = 9; sp.first = i; sp.count = 2; sp.ops = {i, i + 1};
+    sp.keep = {i};                                        // runs of many rows take the two ops one after the other
+    return true;
+}
+
 std::vector<Span> g_spans;
 float* g_attn_scratch = nullptr;
 std::map<std::pair<uint32_t, uint64_t>, uint8_t*> g_skip_maps;   // (mask slot, S<<32|Sk) -> device tile-skip bitmap
@@ -584,6 +602,10 @@ void fuse_analyze(const wt_blob* b, const std::vector<PlanOp>& meas, std::vector
     for (uint32_t i = 0; i + 1 < b->n_ops; i++) {
         Span sp{};
         if (!taken[i] && !taken[i + 1] && match_add_norm(G, i, sp)) claim(sp);
+    }
+    for (uint32_t i = 0; i + 1 < b->n_ops; i++) {
+        Span sp{};
+        if (!taken[i] && !taken[i + 1] && match_latent_step(G, i, sp)) claim(sp);
     }
     // temps written only by interior ops of chains
     std::vector<int> writes_in(kMaxTemps, 0), writes_out(kMaxTemps, 0);
@@ -653,7 +675,20 @@ void fuse_materialize(const wt_blob* b) {
     g.fused_ops = 0;
     for (const Span& sp : g_spans) {
         PlanOp& head = g.plan[sp.first];
-        if (sp.kind == 0) {
+        if (sp.kind == 9) {
+            const PlanOp &ap = g.plan[sp.first], &at = g.plan[sp.first + 1];
+            if (!ap.launch || !at.launch) continue;
+            LatentArgs l = at.rows_args->lat;
+            const LatentArgs& x = ap.rows_args->lat;
+            l.y = x.y; l.norm_w = x.norm_w; l.rope = x.rope; l.eps = x.eps;
+            auto append = ap.launch, attend = at.launch;
+            head.fused = [=](cudaStream_t st) {
+                // few rows: queries taken into latent space, every cached row read once for all heads
+                if (k_latent_step(st, l, rows_of(l.rows_arg))) return;
+                append(st);
+                attend(st);
+            };
+        } else if (sp.kind == 0) {
             const uint16_t* qkv = (const uint16_t*)resolve(b, sp.qkv);
             const uint16_t *cq = (const uint16_t*)resolve(b, sp.cos_q), *sq = (const uint16_t*)resolve(b, sp.sin_q);
             const uint16_t *ck = (const uint16_t*)resolve(b, sp.cos_k), *sk = (const uint16_t*)resolve(b, sp.sin_k);

@@ -16,109 +16,11 @@
 // executor (kernels/src/runtime/oplist_exec.c, cited at each case).
 #include <cstdio>
 #include <cstring>
-#include "engine.h"
+#include "planner.h"
 
 namespace gehtp {
 
 namespace {
-
-struct LiveRange { uint32_t w, r; };  // written at op w, last read at op r
-
-struct Planner {
-    const wt_blob* b;
-    bool build;
-    uint32_t opi = 0;
-    bool written[kMaxTemps];
-    // 64-bit: a temp that only exists inside a fused chain may exceed the 4 GB a
-    // materialised temp is limited to (e.g. the GQA-expanded K/V faces at batch 64)
-    uint64_t cap[kMaxTemps], last[kMaxTemps];
-    // measuring walk results
-    uint64_t maxb[kMaxTemps];
-    bool oversize[kMaxTemps];
-    std::vector<LiveRange> live[kMaxTemps];
-    // building walk inputs
-    uint8_t* addr[kMaxTemps];
-    bool in_static[kMaxTemps], in_vtcm[kMaxTemps];
-    bool internal[kMaxTemps];   // exists only inside fused chains: no memory
-    PlanOp* cur = nullptr;
-
-    uint8_t* dummy() const { return (uint8_t*)(uintptr_t)256; }
-
-    const uint8_t* slot_ptr(uint32_t s) const {
-        if (s >= b->n_slots) return nullptr;
-        const wt_slot& sl = b->slots[s];
-        if (sl.addr == WT_SLOT_EXT_IN || sl.addr == WT_SLOT_EXT_WGT) {
-            if (sl.addr == WT_SLOT_EXT_WGT && !g.ext_wgt) return nullptr;
-            if (!build) return dummy();
-            auto it = g.d_ext.find(s);
-            return it == g.d_ext.end() ? nullptr : it->second;
-        }
-        return build ? g.d_weights + sl.offset : dummy();
-    }
-
-    // ref_ptr, oplist_exec.c:189-203
-    const uint8_t* ref(uint32_t arg) {
-        if (arg & 0x8000u) return slot_ptr(arg & 0x7FFFu);
-        if ((arg & 0xE000u) == WT_REF_STATE_FLAG) {
-            uint32_t s = arg & 0x1FFFu;
-            return s < g.n_states ? g.st_buf[s] : nullptr;
-        }
-        uint32_t t;
-        if (arg & 0x4000u) {
-            t = arg & 0x3FFFu;
-            if (t >= kMaxTemps || g.vtcm_off[t] == kNoOff) return nullptr;
-            if (!build) { touch(t); return dummy(); }
-            return g.d_arena + g.vtcm_base + g.vtcm_off[t];
-        }
-        t = arg;
-        if (t >= kMaxTemps || !written[t]) return nullptr;
-        touch(t);
-        if (build && internal[t]) { if (cur) cur->uses_internal = true; return dummy(); }
-        return build ? addr[t] : dummy();
-    }
-    void touch(uint32_t t) {
-        if (!build && !live[t].empty()) live[t].back().r = opi;
-    }
-    // ref_elem_count, oplist_exec.c:209-213
-    uint32_t ref_count(uint32_t arg) const {
-        if (arg & 0x8000u) { uint32_t s = arg & 0x7FFFu; return s < b->n_slots ? b->slots[s].count : 0; }
-        if (arg & 0x4000u) return 0;
-        return arg < kMaxTemps ? (uint32_t)(last[arg] / 2u) : 0;
-    }
-    // temp_get, oplist_exec.c:257-335
-    uint8_t* temp_get(uint32_t id, uint64_t bytes64, PlanOp& p) {
-        if (id >= kMaxTemps || bytes64 > (1ull << 40)) return nullptr;
-        // Above 4 GB (the reference's temp sizes are 32-bit) only as a temp that fusion removes.
-        if (bytes64 > 0xFFFFFFFFull) {
-            if (!build) oversize[id] = true;
-            else if (!internal[id]) return nullptr;
-        }
-        const uint64_t bytes = bytes64;
-        bool vt = g.vtcm_off[id] != kNoOff, stc = !vt && g.have_static && g.static_off[id] != kNoOff;
-        if (vt && (uint64_t)g.vtcm_off[id] + bytes > g.vtcm_cap) return nullptr;
-        if (stc && (!build || in_static[id]) && (uint64_t)g.static_off[id] + bytes > g.static_cap) return nullptr;
-        if (vt || stc) cap[id] = bytes;
-        else if (!written[id] || cap[id] < bytes) cap[id] = bytes;
-        last[id] = bytes;
-        written[id] = true;
-        for (int k = 0; k < 2; k++)
-            if (p.out_id[k] == kNoOff || p.out_id[k] == id) { p.out_id[k] = id; p.out_bytes[k] = (uint32_t)(bytes > 0xFFFFFFFFull ? 0xFFFFFFFFull : bytes); break; }
-        if (!build) {
-            if (bytes > maxb[id]) maxb[id] = bytes;
-            live[id].push_back({opi, opi});
-            return dummy();
-        }
-        if (internal[id]) { p.uses_internal = true; return dummy(); }
-        return addr[id];
-    }
-};
-
-#define FAIL(...)                                            \
-    do {                                                     \
-        char _m[160];                                        \
-        std::snprintf(_m, sizeof _m, __VA_ARGS__);           \
-        p.rc = -1; p.err = _m; return;                       \
-    } while (0)
 
 // KV ring geometry of a state, derived from the op's K/V width on first use
 // (state_kvc, oplist_exec.c:2119-2151).
@@ -683,6 +585,7 @@ void plan_op(Planner& P, const wt_op& op, PlanOp& p) {
         return;
     }
     default:
+        if (op.opcode >= OP_EMBED_ROWS && op.opcode < OP_ROWS_END) { plan_rows_op(P, op, p); return; }
         FAIL("opcode %u unhandled", (unsigned)op.opcode);
     }
 }
@@ -778,6 +681,23 @@ int load_states(const wt_blob* b, char* err, size_t errn) {
     return 0;
 }
 
+// ROWS table: {max_rows, max_sel} of a row-count runlist; absent: both 0.
+int load_rows(const wt_blob* b, char* err, size_t errn) {
+    g.max_rows = g.max_sel = 0;
+    for (uint32_t s = 0; s < b->n_slots; s++) {
+        if (b->slots[s].addr != WT_SLOT_ROWS) continue;
+        const uint8_t* p = b->weight_base + b->slots[s].offset;
+        if (b->slots[s].len < 8u) { std::snprintf(err, errn, "rows slot short"); return -1; }
+        g.max_rows = wt_rd_u32(p);
+        g.max_sel = wt_rd_u32(p + 4);
+        if (!g.max_rows || !g.max_sel || g.max_sel > g.max_rows) { std::snprintf(err, errn, "rows slot bad (%u, %u)", g.max_rows, g.max_sel); return -1; }
+        break;
+    }
+    g.run_rows = g.max_rows;
+    g.run_sel = g.max_sel;
+    return 0;
+}
+
 bool ranges_clash(const std::vector<LiveRange>& x, const std::vector<LiveRange>& y) {
     for (const auto& a : x)
         for (const auto& c : y)
@@ -794,6 +714,7 @@ int build_plan(const wt_blob* b, char* err, size_t errn) {
     if (!err) { err = scratch; errn = sizeof scratch; }
     if (load_tempoff(b, err, errn) != 0) return -1;
     if (load_states(b, err, errn) != 0) return -1;
+    if (load_rows(b, err, errn) != 0) return -1;
 
     // device copies of the slot data
     if (b->weight_bytes) {
@@ -912,9 +833,9 @@ int build_plan(const wt_blob* b, char* err, size_t errn) {
 }
 
 void drop_plan(bool keep_states) {
-    if (g.graph) { cudaGraphExecDestroy(g.graph); g.graph = nullptr; }
+    drop_graphs();
     g.plan.clear();
-    g.planned = false; g.blob = nullptr; g.warm_runs = 0;
+    g.planned = false; g.blob = nullptr; g.warm_runs.clear();
     if (g.d_weights) { cudaFree(g.d_weights); g.d_weights = nullptr; }
     for (auto& kv : g.d_ext) cudaFree(kv.second);
     g.d_ext.clear();

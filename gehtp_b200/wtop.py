@@ -14,6 +14,11 @@ import numpy as np
 WT_MAX_SLOTS, WT_MAX_OPS, WT_MAX_ARGS = 4096, 65536, 16
 SLOT_EXT_IN, SLOT_EXT_OUT, SLOT_TEMPOFF = 0xFFFFFFFF, 0xFFFFFFFE, 0xFFFFFFFD
 SLOT_EXT_WGT, SLOT_STATE, KV_POS_AUTO = 0xFFFFFFFC, 0xFFFFFFFB, 0xFFFFFFFA
+# row-count runlists (this executor's own): limits slot, and the row arguments that follow the run
+SLOT_ROWS, ROWS_AUTO, SEL_AUTO = 0xFFFFFFF7, 0xFFFFFFF9, 0xFFFFFFF8
+DT_F32, DT_BF16 = 0, 1
+LIN_X_BF16, LIN_Y_BF16, LIN_RELU2 = 1, 2, 16
+COL_ALIGN = 8
 
 
 class OP:
@@ -22,17 +27,22 @@ class OP:
     CONV1D_SSM, GATHER, ARGMAX, KV_APPEND, KV_GATHER, MATMUL_F16, RMSNORM2 = range(19, 26)
     BROADCAST, TRANSPOSE_GEN, SCATTER_ND, CONV1D_SSM_STEP, DELTA_CHUNK = range(26, 31)
     DMA, PAD, MATMUL_F16_SPLIT = 33, 34, 35
+    EMBED_ROWS, LINEAR, NORM_RESID, PICK_ROWS, LATENT_APPEND, LATENT_ATTEND = range(0x140, 0x146)
+    SHORT_CONV, CHANNEL_DELTA, GATED_NORM, ARGMAX_ROWS, STATE_ADVANCE = range(0x146, 0x14B)
 
 
 ARITY = {0: 0, 1: 6, 2: 4, 3: 1, 4: 3, 5: 15, 6: 13, 7: 4, 8: 4, 9: 4, 10: 6, 11: 4, 12: 5, 13: 4,
          14: 16, 15: 16, 16: 16, 17: 9, 18: 7, 19: 6, 20: 15, 21: 3, 22: 4, 23: 7, 24: 7, 25: 5,
-         26: 12, 27: 8, 28: 14, 29: 6, 30: 12, 33: 8, 34: 7, 35: 9}
+         26: 12, 27: 8, 28: 14, 29: 6, 30: 12, 33: 8, 34: 7, 35: 9,
+         0x140: 8, 0x141: 9, 0x142: 9, 0x143: 6, 0x144: 13, 0x145: 14, 0x146: 9, 0x147: 16, 0x148: 9, 0x149: 4, 0x14A: 3}
 
 
 # argument positions that name the temp(s) an op writes
 _OUT_ARGS = {1: (2,), 4: (1,), 7: (2,), 10: (1,), 11: (1,), 12: (2,), 13: (1,), 14: (8,), 15: (1,), 16: (1,),
              17: (1,), 18: (1,), 19: (2,), 20: (2,), 21: (1,), 23: (1, 2), 24: (2,), 25: (3,), 26: (1,),
-             27: (1,), 28: (3,), 29: (2,), 30: (5,), 34: (1,), 35: (2,)}
+             27: (1,), 28: (3,), 29: (2,), 30: (5,), 34: (1,), 35: (2,),
+             0x140: (2, 3), 0x141: (2,), 0x142: (3, 4), 0x143: (3,), 0x144: (3, 4), 0x145: (4, 5), 0x146: (3,), 0x147: (6, 7),
+             0x148: (3,), 0x149: (1,)}
 
 
 def op_out_temps(op):
@@ -101,6 +111,10 @@ class BlobBuilder:
 
     def add_states(self, sizes):
         return self.add_slot(struct.pack("<I%dI" % len(sizes), len(sizes), *sizes), addr=SLOT_STATE)
+
+    def add_rows(self, max_rows, max_sel):
+        """Makes the blob a row-count runlist: up to max_rows token rows per run, max_sel of them picked for the head."""
+        return self.add_slot(struct.pack("<II", max_rows, max_sel), addr=SLOT_ROWS)
 
     def add_tempoff(self, cap, entries, bump_kb=0, vtcm_kb=0):
         """entries: (temp_id, offset, size); temp_id may carry 0x4000 for the on-chip region."""
@@ -205,6 +219,7 @@ def bind(lib):
         lib.gehtp_cuda_set_device.argtypes = [c.c_int]
         lib.gehtp_cuda_set_fusion.argtypes = [c.c_int]
         lib.gehtp_cuda_set_graph.argtypes = [c.c_int]
+        lib.gehtp_cuda_set_rows.argtypes = [P(WtBlob), c.c_uint32, c.c_uint32, c.c_char_p, c.c_size_t]
         lib.gehtp_cuda_run_dev.argtypes = [P(WtBlob), c.c_void_p, c.c_void_p, c.c_uint32, c.c_char_p, c.c_size_t]
         lib.gehtp_cuda_run_profiled.argtypes = [P(WtBlob), c.c_void_p, c.c_uint32, P(c.c_float), c.c_uint32, c.c_char_p, c.c_size_t]
         lib.gehtp_cuda_profiled_attn.argtypes = [P(c.c_float), P(c.c_uint32)]
@@ -277,6 +292,10 @@ class Engine:
 
     def run_range(self, first, count):
         self._check(self.lib.wt_exec_run_range(ctypes.byref(self.blob), first, count, None, None, self._err, 256))
+
+    def set_rows(self, rows, sel):
+        """Token rows of the next runs of a row-count runlist, and how many of them are picked for the head."""
+        self._check(self.lib.gehtp_cuda_set_rows(ctypes.byref(self.blob), rows, sel, self._err, 256))
 
     def run_io(self, inp, out_temp, out=None):
         """inp: numpy array or None; out: preallocated numpy array or None. Returns out."""

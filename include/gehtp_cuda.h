@@ -118,6 +118,12 @@ void gehtp_cuda_set_fusion(int on);
  * force eager execution for that run. */
 void gehtp_cuda_set_graph(int on);
 
+/* Row-count runlists (WT_SLOT_ROWS): the next runs of `b` process `rows` token rows, `sel` of which are picked for
+ * the head (0: no head output). Plans the blob if it is not planned yet; before the first call the largest counts of
+ * the blob apply. The input face always has its full size; temps whose size follows a count report the bytes of the
+ * last run through wt_exec_temp_last_bytes. Returns 0, or -1 (counts beyond the blob's, or not such a blob). */
+int gehtp_cuda_set_rows(const struct wt_blob* b, uint32_t rows, uint32_t sel, char* err, size_t errn);
+
 /* Tensor parallelism inside one node: this process is `rank` of `world`.
  * `nccl_unique_id` is the 128-byte id made by rank 0 and sent to the others by
  * the caller (the engine does no rendezvous of its own). Column- and

@@ -54,6 +54,13 @@ extern "C" {
 #define WT_SLOT_STATE      0xFFFFFFFBu  /* persistent state size table            */
 #define WT_KV_POS_AUTO     0xFFFFFFFAu  /* KV pos / n_kv taken from state counter */
 
+/* Row-count runlists (no counterpart in the reference). A blob with a WT_SLOT_ROWS slot - u32 {max_rows, max_sel} -
+ * may be run with any number of token rows up to max_rows, of which up to max_sel are picked for the head
+ * (gehtp_cuda_set_rows). Row arguments of the ops below take these markers instead of a number. */
+#define WT_SLOT_ROWS       0xFFFFFFF7u
+#define WT_ROWS_AUTO       0xFFFFFFF9u  /* token rows of the run                     */
+#define WT_SEL_AUTO        0xFFFFFFF8u  /* rows picked for the head in this run      */
+
 #define WT_REF_SLOT_FLAG   0x8000u
 #define WT_REF_VTCM_FLAG   0x4000u
 #define WT_REF_STATE_FLAG  0x6000u
@@ -77,6 +84,43 @@ enum {
     OP_CONV1D_SSM_STEP_F16 = 29, OP_DELTA_CHUNK_F16 = 30,
     OP_DMA = 33, OP_PAD_F16 = 34, OP_MATMUL_F16_SPLIT = 35
 };
+
+/* Opcodes of this executor alone, far from the reference's numbers. Activations are bf16 or fp32 (WT_DT_*), weights
+ * bf16 as stored in checkpoints, the residual stream, norms, gates, scores and recurrent state fp32.
+ * "rows" arguments: a number, WT_ROWS_AUTO or WT_SEL_AUTO. Sizes are in elements, *_bits are fp32 bit patterns.
+ *
+ * OP_EMBED_ROWS     [table, ids, x_out, act_out, rows, width, vocab, dt]      x = table[id] (fp32), act = x in dt
+ * OP_LINEAR         [x, w, y, rows, K, N, flags, x_col, x_stride]             y = act(x[:, x_col: x_col + K] . w^T), w bf16 [N, K];
+ *                   flags: WT_LIN_*; x_stride 0 = K
+ * OP_NORM_RESID     [y, w, x, x_out, act_out, rows, width, flags, eps_bits]   x_out = x + y / rms(y) * (b + w), w fp32;
+ *                   flags: bit 0 b = 1 (weight stored around zero) else b = 0, bit 1 act_out is bf16, bit 2 y is bf16.
+ *                   x = 0: no residual; x_out / act_out = 0: not written
+ * OP_PICK_ROWS      [x, idx, idx_off, out, rows, width]                       out[r] = x[idx[idx_off + r]] (fp32 rows, int32 idx)
+ * OP_LATENT_APPEND  [y, norm_w, rope, q_out, gate_out, state, rows, heads, dim, rot, rank, eps_bits, flags]
+ *                   y rows = [q: heads x (dim | rot) | latent: rank | key part: rot | gate: heads], each group starting at a
+ *                   multiple of 8; rope: fp32 [positions][rot / 2][cos, sin], neighbouring components paired. Appends
+ *                   [norm(latent) * norm_w | rotated key part] to the state at the state's position counter; flags: WT_DT_*
+ * OP_LATENT_ATTEND  [q, gate, state, w_kv, out, work, rows, heads, dim, rot, vdim, rank, scale_bits, flags]
+ *                   w_kv bf16 = [up-projection of keys: heads x dim | of values: heads x vdim][rank]; causal over the state;
+ *                   out = softmax(q . k * scale) v * sigmoid(gate) per head; work: scratch temp
+ * OP_SHORT_CONV     [y, w, state, out, rows, channels, taps, y_stride, flags] out = silu(causal depthwise conv of y[:, :channels]),
+ *                   w fp32 [channels][taps], last tap = current token; fp32 out, the last taps - 1 inputs live in the state
+ * OP_CHANNEL_DELTA  [qkv, a, y, a_log, dt_bias, state, out, work, rows, heads, kv_heads, dim, vdim, b_col, y_stride, flags]
+ *                   delta rule with a decay per key channel: S <- exp(-exp(a_log) softplus(a + dt_bias)) S,
+ *                   u = sigmoid(b)(v - S^T k), S <- S + k u^T, out = S^T q; q, k unit vectors, q * dim^-1/2
+ * OP_GATED_NORM     [o, w, gate, out, rows, heads, vdim, eps_bits, flags]     out = o / rms(o) * w * sigmoid(gate) per head
+ * OP_ARGMAX_ROWS    [x, out, rows, n]                                         int32 per row of fp32 x
+ * OP_STATE_ADVANCE  [first, n, rows]                                          adds rows to the position counters of n states */
+enum {
+    OP_EMBED_ROWS = 0x140, OP_LINEAR, OP_NORM_RESID, OP_PICK_ROWS, OP_LATENT_APPEND, OP_LATENT_ATTEND, OP_SHORT_CONV,
+    OP_CHANNEL_DELTA, OP_GATED_NORM, OP_ARGMAX_ROWS, OP_STATE_ADVANCE, OP_ROWS_END
+};
+#define WT_DT_F32   0u
+#define WT_DT_BF16  1u
+#define WT_LIN_X_BF16  1u
+#define WT_LIN_Y_BF16  2u
+#define WT_LIN_RELU2   16u   /* y = max(x . w, 0)^2 */
+#define WT_COL_ALIGN   8u    /* column groups of a joined projection start at multiples of this many elements */
 
 /* Fixed argument count per opcode (oplist_parse.h:218-251). */
 #define WT_ARITY_NOP 0
