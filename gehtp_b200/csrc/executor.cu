@@ -54,7 +54,11 @@ bool ensure_device(char* err, size_t errn) {
 
 static void grow_pinned(uint8_t*& p, size_t& cap, size_t need) {
     if (need <= cap) return;
-    if (p) cudaFreeHost(p);
+    if (p) {
+        cudaStreamSynchronize(g.stream);
+        drop_graphs();          // captured copies carry the old address
+        cudaFreeHost(p);
+    }
     cap = (need + 4095) / 4096 * 4096;
     if (cudaMallocHost(&p, cap) != cudaSuccess) { p = nullptr; cap = 0; }
 }
@@ -505,7 +509,7 @@ static int run_impl(const wt_blob* b, uint32_t first, uint32_t count, const void
     if (out_dev && out_temp < kMaxTemps && g.temp_cap[out_temp])
         cudaMemcpyAsync(out_dev, g.temp_dev[out_temp], g.temp_last[out_temp], cudaMemcpyDeviceToDevice, g.stream);
     if (out_host && out_temp < kMaxTemps && g.temp_cap[out_temp]) {
-        grow_pinned(g.h_out, g.h_out_cap, g.temp_last[out_temp]);
+        grow_pinned(g.h_out, g.h_out_cap, g.temp_cap[out_temp]);
         cudaMemcpyAsync(g.h_out, g.temp_dev[out_temp], g.temp_last[out_temp], cudaMemcpyDeviceToHost, g.stream);
     }
     if (!sync_end) return 0;
