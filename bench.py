@@ -49,6 +49,10 @@ def parse_args():
                          "3: 0.6B-shape prefill, 5: gated delta-rule layer) with its roofline and the reference's CPU time")
     ap.add_argument("--micro", default=None, choices=["gemv", "lmhead", "gemm", "swiglu", "swiglu512", "gemm1", "gemm512", "f16gemm", "headline", "gemmtiles", "attn", "attn8", "norm", "prefill", "gdn", "all"],
                     help="time single kernels (device-resident operands, graph replay) instead of the decode step")
+    ap.add_argument("--design", default=None, choices=["Ripidra"],
+                    help="prefill and decode of a model design at real layer sizes (random weights), beside the decoder of the same width, "
+                         "feed-forward and heads with fp16 weights: tokens/s and, per launch unit, time against its roofline")
+    ap.add_argument("--sizes", default="1024,2560", help="widths for --design, with commas between them")
     return ap.parse_args()
 
 
@@ -842,6 +846,215 @@ def run_config(args):
     return line
 
 
+# widths of --design: (feed-forward, heads); both designs get heads of 128
+DESIGN_SIZES = {1024: (3072, 16), 2560: (9728, 32)}
+
+
+def design_model(width, vocab):
+    """A Ripidra model of 2 latent-attention and 2 channel-delta layers with random weights (a 1M-value block, tiled)."""
+    from gehtp_b200.checkpoint import ArrayTensors, f32_to_bf16
+    from gehtp_b200.registry import Model
+    ff, H = DESIGN_SIZES[width]
+    lat = dict(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=512, rot=dict(base=1e6, dims=64), scale=192 ** -0.5)
+    dlt = dict(heads=H, kv_heads=H, dim=128, vdim=128, conv=4)
+    kinds = [("channel_delta", dlt), ("latent_attention", lat)] * 2
+    cfg = dict(architecture="Ripidra", vocab=vocab, width=width, norm=dict(eps=1e-6),
+               layers=[dict(type=k, mixer=m, mlp=dict(kind="dense", ff=ff)) for k, m in kinds])
+    block = np.random.default_rng(9).standard_normal(1 << 20, dtype=np.float32)
+
+    def mat(n, k, scale=None):
+        b = f32_to_bf16(block * np.float32(k ** -0.5 if scale is None else scale))
+        return np.resize(b, (n, k)) if k else np.resize(b, n)
+    t = {"embed": mat(vocab, width, 1.0), "final.norm": mat(width, 0, 0.1)}
+    for i, (k, m) in enumerate(kinds):
+        p = "l%d." % i
+        t[p + "norm1"], t[p + "norm2"] = mat(width, 0, 0.1), mat(width, 0, 0.1)
+        t[p + "mlp.up"], t[p + "mlp.down"] = mat(ff, width), mat(width, ff)
+        q = p + "mix."
+        if k == "latent_attention":
+            t.update({q + "q": mat(H * 192, width), q + "dkv": mat(576, width), q + "dkv.norm": mat(512, 0, 1.0), q + "uk": mat(H * 128, 512),
+                      q + "uv": mat(H * 128, 512), q + "g": mat(H, width), q + "o": mat(width, H * 128)})
+        else:
+            for n in "qkv":
+                t[q + n], t[q + n + ".conv"] = mat(H * 128, width), mat(H * 128, 4, 0.5)
+            t.update({q + "b": mat(H, width), q + "A_log": mat(H, 0, 0.5), q + "norm": mat(128, 0, 1.0), q + "a1": mat(128, width),
+                      q + "a2": mat(H * 128, 128), q + "dt_bias": mat(H * 128, 0, 1.0), q + "g1": mat(128, width), q + "g2": mat(H * 128, 128),
+                      q + "o": mat(width, H * 128)})
+    return Model(cfg, ArrayTensors(t))
+
+
+def run_design(args, width):
+    """One line per (design, phase): tokens/s of the run by events on the engine stream, and the launch units of one
+    profiled run with their algorithmic work. Prefill: 2048 tokens from position 0; decode: one token at context 8192."""
+    import torch
+    import gehtp_b200
+    from gehtp_b200.runlists import DecoderConfig, build_decode_runlist, build_prefill_runlist, decode_face
+    from gehtp_b200.session import Session
+    from gehtp_b200.wtop import OP, ROWS_AUTO, SEL_AUTO, Engine
+    lib = gehtp_b200.lib()
+    assert lib.gehtp_cuda_set_device(0) == 0, "no CUDA device"
+    pk = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = float(pk.get("hbm_gbs", 6650.0)), float(pk.get("bf16_tflops", 1590.0))
+    stream = torch.cuda.ExternalStream(lib.gehtp_cuda_stream())
+    err = ctypes.create_string_buffer(256)
+    S_, CTX, V = 2048, 8192, 32768
+    ff, H = DESIGN_SIZES[width]
+    K, W = args.steps, max(args.warmup, 3)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def timed(step, rewind=lambda: None):
+        """Mean of K steps, each timed on its own after L2 has been overwritten."""
+        for _ in range(W):
+            rewind()
+            step()
+        tot = 0.0
+        for _ in range(K):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            rewind()
+            with torch.cuda.stream(stream):
+                flush.zero_()
+                e0.record()
+            step()
+            with torch.cuda.stream(stream):
+                e1.record()
+            torch.cuda.synchronize()
+            tot += e0.elapsed_time(e1)
+        return tot / K
+
+    def units(eng, face, out_temp, work):
+        """Launch units of one profiled run: name -> launches, us, and the fraction of the roofline time."""
+        ms = (ctypes.c_float * eng.blob.n_ops)()
+        assert lib.gehtp_cuda_run_profiled(ctypes.byref(eng.blob), face.ctypes.data, out_temp, ms, eng.blob.n_ops, err, 256) == 0, err.value
+        acc = {}
+        for i in range(eng.blob.n_ops):
+            if ms[i] <= 0:
+                continue
+            name, by, fl = work(i, eng.blob.ops[i])
+            u = acc.setdefault(name, [0, 0.0, 0.0])
+            u[0] += 1
+            u[1] += ms[i] * 1e3
+            u[2] += max(by / hbm / 1e3, fl / tf / 1e6)
+        return {n: {"launches": c, "us": round(us / c, 2), "roofline_us": round(r / c, 2), "frac": round(r / us, 3)} for n, (c, us, r) in sorted(acc.items())}
+
+    lines = []
+    clocks = None
+
+    def add(design, phase, ms, tokens, un):
+        lines.append({"design": design, "width": width, "ff": ff, "heads": H, "layers": 4, "phase": phase, "ms": round(ms, 4),
+                      "tok_s": round(tokens / ms * 1e3, 1), "units": un, "clocks": clocks, "l2": "overwritten before every timed step"})
+
+    # ---- the design
+    s = Session(design_model(width, V), max_tokens=CTX, max_rows=S_, max_sel=16)
+    eng, man = s.engine, s.man
+    rng = np.random.default_rng(5)
+
+    def work_rows(rows, past):
+        def f(i, op):
+            a = list(op.args)
+            n = rows if ROWS_AUTO in a else 1
+            if op.opcode == OP.LINEAR:
+                r = 1 if a[3] == SEL_AUTO else rows
+                k, c = a[4], a[5]
+                yb = 2 if a[6] & 2 else 4
+                return "linear %dx%d" % (k, c), 2 * k * c + r * (2 * k + yb * c), 2.0 * r * k * c
+            if op.opcode in (OP.LATENT_APPEND, OP.LATENT_ATTEND):
+                ctx = past + rows
+                if rows > 16 and op.opcode == OP.LATENT_APPEND:
+                    return "latent append + attend", 2 * rows * (H * 192 * 2 + 576), 2.0 * ctx * 512 * H * 256 + 2.0 * H * 320 * rows * (past + rows / 2)
+                return "latent append + attend", ctx * 576 * 2 + H * 256 * 512 * 2, 2.0 * rows * H * (256 * 512 + ctx * 1088)
+            if op.opcode == OP.SHORT_CONV:
+                return "short conv .. gated norm" if rows <= 8 else "short conv", rows * 3 * H * 128 * 6, 0
+            if op.opcode == OP.CHANNEL_DELTA:
+                return "channel delta", rows * H * 128 * 4 * 6 + H * 128 * 128 * 8, 0
+            if op.opcode == OP.GATED_NORM:
+                return "gated norm", rows * H * 128 * 10, 0
+            if op.opcode == OP.NORM_RESID:
+                return "norm + residual", n * width * 14, 0
+            return "other", 0, 0
+        return f
+
+    def phase(rows, ctx, name):
+        face = np.zeros(man["max_rows"] + man["max_sel"], np.int32)
+        face[:rows] = rng.integers(0, V, rows)
+        face[man["max_rows"]] = rows - 1
+        dface = torch.from_numpy(face).cuda()
+        out = torch.zeros(4, dtype=torch.int32, device="cuda")
+        s.reset()
+        for p in range(0, ctx, S_):
+            s.feed(rng.integers(0, V, min(S_, ctx - p)), [])
+        eng.set_rows(rows, 1)
+
+        def rewind():
+            for i in range(2):
+                assert lib.gehtp_cuda_state_set_count(i, ctx) == 0
+
+        def step():
+            assert lib.gehtp_cuda_run_dev(ctypes.byref(eng.blob), dface.data_ptr(), out.data_ptr(), man["token_temp"], err, 256) == 0, err.value
+        ms = timed(step, rewind)
+        rewind()
+        un = units(eng, face, man["token_temp"], work_rows(rows, ctx))
+        add(args.design, name, ms, rows, un)
+
+    sampler = ClockSampler(0)
+    sampler.start()
+    phase(S_, 0, "prefill 2048")
+    phase(1, CTX - 64, "decode ctx %d" % (CTX - 64))
+    s.close()
+    clocks = sampler.stop()
+    for ln in lines:
+        ln["clocks"] = clocks
+
+    # ---- the decoder of the same width with fp16 weights
+    cfg = DecoderConfig(width, 4, H, 8, 128, ff, V, 1e6, "decoder-%d" % width)
+    buf, man = build_prefill_runlist(cfg, S_, quant="f16", with_lm_head=False)
+    eng = Engine(lib, buf)
+
+    def work_fixed(rows, ctx):
+        def f(i, op):
+            a = list(op.args)
+            if op.opcode == OP.MATMUL_F16 and not a[6] & 4:
+                return "linear %dx%d" % (a[4], a[5]), 2 * (a[4] * a[5] + rows * (a[4] + a[5])), 2.0 * rows * a[4] * a[5]
+            if op.opcode in (OP.SPLIT, OP.TRANSPOSE_GEN, OP.MATMUL_F16):
+                if rows > 1 and op.opcode == OP.SPLIT:
+                    return "split + rotary", rows * (H + 16) * 128 * 4, 0
+                if rows > 1:
+                    return "attention", 0, 4.0 * H * 128 * rows * rows / 2
+                return "attention", 2 * ctx * 8 * 128 * 2, 4.0 * H * 128 * ctx
+            if op.opcode == OP.RMSNORM2 or op.opcode == OP.ADD:
+                return "add + norm", rows * width * 8, 0
+            return "other", 0, 0
+        return f
+    ids = rng.integers(0, V, S_).astype(np.int32)
+    dids = torch.from_numpy(ids).cuda()
+    hid = torch.zeros(S_ * width, dtype=torch.int16, device="cuda")
+
+    def step():
+        assert lib.gehtp_cuda_run_dev(ctypes.byref(eng.blob), dids.data_ptr(), hid.data_ptr(), man["hidden_temp"], err, 256) == 0, err.value
+    ms = timed(step)
+    add(cfg.name, "prefill 2048", ms, S_, units(eng, ids, man["hidden_temp"], work_fixed(S_, S_)))
+    eng.shutdown()
+    buf, man = build_decode_runlist(cfg, 1, CTX, quant="f16")
+    eng = Engine(lib, buf)
+    for li in range(4):
+        kv = torch.randn(CTX * 2 * 1024, device="cuda", dtype=torch.float16)
+        assert lib.gehtp_cuda_state_load(ctypes.byref(eng.blob), li, kv.data_ptr(), kv.numel() * 2, 1, 1024, CTX - 64, err, 256) == 0, err.value
+    face = decode_face(man, [7], CTX - 64, 128, 1e6)
+    dface = torch.from_numpy(face.view(np.int16).copy()).cuda()
+    out = torch.zeros(4, dtype=torch.int16, device="cuda")
+
+    def rewind():
+        for li in range(4):
+            assert lib.gehtp_cuda_state_set_count(li, CTX - 64) == 0
+
+    def step():
+        assert lib.gehtp_cuda_run_dev(ctypes.byref(eng.blob), dface.data_ptr(), out.data_ptr(), man["token_temp"], err, 256) == 0, err.value
+    ms = timed(step, rewind)
+    rewind()
+    add(cfg.name, "decode ctx %d" % (CTX - 64), ms, 1, units(eng, face, man["token_temp"], work_fixed(1, CTX)))
+    eng.shutdown()
+    return lines
+
+
 def _op_work(opcode, a):
     """Scalar operations of one op record, for scaling a reference timing to another sequence length."""
     from gehtp_b200.wtop import OP
@@ -1000,6 +1213,12 @@ def run_main(args):
                              ("single GPU" if args.shard_of <= 1 else "rank 0's shard of tp%d, no all-reduce (profiling aid)" % args.shard_of),
               "l2": "inputs larger than L2: every step streams the weights and the KV rings (GBs) once"}
 
+    if args.design:
+        if rank == 0:
+            for w in args.sizes.split(","):
+                for row in run_design(args, int(w)):
+                    out.append(json.dumps(row))
+        return out
     if args.micro:
         if rank == 0:
             for row in run_micro(args.micro):

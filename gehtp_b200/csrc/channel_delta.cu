@@ -4,12 +4,14 @@
 //                        a run reads the bank of its parity and writes the other, so that no CTA overwrites what
 //                        another still reads
 //   delta_prep_kernel    unit vectors, decays, step sizes, k . q per token, fp32
-//   delta_scan_kernel    the recurrence, token by token: a column of S lives in the registers of 8 (16, 32) lanes, both
-//                        reductions of a token (S^T k and S^T q) run side by side; with S' = g S,
-//                        u = beta (v - S'^T k), S = S' + k u^T:  S^T q = S'^T q + u (k . q)
+//   delta_scan_kernel    the recurrence, token by token: S lives in registers, 2 columns per 16 lanes, both reductions of
+//                        a token (S^T k and S^T q) run side by side; with S' = g S, u = beta (v - S'^T k),
+//                        S = S' + k u^T:  S^T q = S'^T q + u (k . q)
 //   gated_norm_kernel    RMS norm of a head's read-out, weight, sigmoid gate
+//   delta_step_kernel    all of it for up to 4 rows, with the second halves of the low-rank decay and gate projections
 //
 // The recurrence is the same arithmetic for one token and for a whole prompt, so a cut of the prompt changes nothing.
+#include <cooperative_groups.h>
 #include "launchers_rows.h"
 #include "mma_bf16.cuh"
 
@@ -112,100 +114,139 @@ delta_prep_kernel(const DeltaArgs a, const DeltaWork wk) {
     }
 }
 
-// LPC lanes hold a column of S, RPL rows each; a warp holds 32 / LPC columns, a CTA 8 warps of one head. Tokens come in
-// chunks of TC through shared memory (cp.async, two stages; VEC = 16-byte copies).
+// two fp32 values side by side (fma.rn.f32x2): the same roundings as two scalar operations
+__device__ __forceinline__ uint64_t pk2(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
+__device__ __forceinline__ float sum2(uint64_t v) { float a, b; asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); return a + b; }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) { uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
+
+// 16 lanes hold 2 neighbouring columns of S, RPL rows each (as RPL / 2 pairs); a warp holds 4 columns, a CTA NW warps of
+// one head. Every value of k, q and g that a lane reads from shared memory serves 2 columns; those of the next token are
+// read while this token's sums are reduced. The four sums of a token (S^T k and S^T q of 2 columns) are reduced over the
+// 16 lanes by halving: an exchange leaves a lane with half of the sums it had, until lane (kind, column, -, -) holds one.
+// Tokens come in chunks of TC through shared memory (cp.async, two stages; VEC = 16-byte copies).
 constexpr uint32_t TC = 16;
-template <int LPC, int RPL, bool VEC>
-__global__ void __launch_bounds__(256)
+template <int RPL, int NW, bool VEC>
+__global__ void __launch_bounds__(NW * 32)
 delta_scan_kernel(const DeltaArgs a, const DeltaWork wk, uint32_t rows) {
-    constexpr uint32_t DP = LPC * RPL, CPW = 32 / LPC, NC = 8 * CPW;
+    constexpr uint32_t DP = 16 * RPL, NC = NW * 4, NT = NW * 32;
     extern __shared__ __align__(16) float sm[];
     float* s_kqg = sm;                                // [2][TC][3][DP]
     float* s_v = s_kqg + 2 * TC * 3 * DP;             // [2][TC][NC]
     float* s_bk = s_v + 2 * TC * NC;                  // [2][TC][2]
-    pdl_release();
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, H = a.heads, D = a.dim, V = a.vdim;
     const uint32_t h = blockIdx.y, kh = h / (H / a.kv_heads), c0 = blockIdx.x * NC;
-    const uint32_t l = lane % LPC, col = c0 + warp * CPW + lane / LPC;
+    const uint32_t l = lane & 15, base = lane & 16, cl = warp * 4 + (lane >> 4) * 2;      // first of this lane's columns, within the CTA
     const uint32_t C = a.channels(), voff = 2 * a.kv_heads * D + h * V;
-    for (uint32_t i = tid; i < 2 * TC * 3 * DP; i += 256)
+    for (uint32_t i = tid; i < 2 * TC * 3 * DP; i += NT)
         if (i % DP >= D) s_kqg[i] = 0.0f;             // rows past D: S stays zero there
-    pdl_wait();
+    for (uint32_t i = tid; i < 2 * TC * NC; i += NT)
+        if (c0 + i % NC >= V) s_v[i] = 0.0f;          // columns past V, which no copy writes
     float* Sg = a.S + (size_t)h * D * V;
-    auto row_of = [&](int i) -> uint32_t { return (i / 4) * 4 * LPC + l * 4 + (i & 3); };
-    float S[RPL];
+    auto row_of = [&](int i) -> uint32_t { return (i / 4) * 64 + l * 4 + (i & 3); };
+    uint64_t S[RPL / 2][2];
 #pragma unroll
-    for (int i = 0; i < RPL; i++) {
+    for (int i = 0; i < RPL; i += 2) {
         const uint32_t r = row_of(i);
-        S[i] = (r < D && col < V) ? Sg[(size_t)r * V + col] : 0.0f;
+#pragma unroll
+        for (int c = 0; c < 2; c++) {
+            const uint32_t col = c0 + cl + c;
+            S[i / 2][c] = pk2((r < D && col < V) ? Sg[(size_t)r * V + col] : 0.0f, (r + 1 < D && col < V) ? Sg[(size_t)(r + 1) * V + col] : 0.0f);
+        }
     }
     auto fetch = [&](uint32_t t0, uint32_t stg) {
         const uint32_t nt = t0 < rows ? min(TC, rows - t0) : 0;
         float* d = s_kqg + stg * TC * 3 * DP;
-        if (VEC) {
-            const uint32_t ch = D / 4;
-            for (uint32_t i = tid; i < nt * 3 * ch; i += 256) {
-                const uint32_t t = i / (3 * ch), w = (i / ch) % 3, c = (i % ch) * 4;
-                const float* src = w == 2 ? wk.g + ((size_t)(t0 + t) * H + h) * D + c
-                                          : (w ? wk.q : wk.k) + ((size_t)(t0 + t) * a.kv_heads + kh) * D + c;
-                cp16(smem_addr(d + (t * 3 + w) * DP + c), src, 16);
+        // warp w copies tokens w, w + NW, ...: k, q and g of a token, lanes along the channels
+        for (uint32_t t = warp; t < nt; t += NW) {
+            const float* sk = wk.k + ((size_t)(t0 + t) * a.kv_heads + kh) * D;
+            const float* sq = wk.q + ((size_t)(t0 + t) * a.kv_heads + kh) * D;
+            const float* sg = wk.g + ((size_t)(t0 + t) * H + h) * D;
+            float* dt = d + t * 3 * DP;
+            if (VEC) {
+                for (uint32_t c = lane * 4; c < D; c += 128) {
+                    cp16(smem_addr(dt + c), sk + c, 16);
+                    cp16(smem_addr(dt + DP + c), sq + c, 16);
+                    cp16(smem_addr(dt + 2 * DP + c), sg + c, 16);
+                }
+            } else {
+                for (uint32_t c = lane; c < D; c += 32) { dt[c] = __ldcg(sk + c); dt[DP + c] = __ldcg(sq + c); dt[2 * DP + c] = __ldcg(sg + c); }
             }
-        } else {
-            for (uint32_t i = tid; i < nt * 3 * D; i += 256) {
-                const uint32_t t = i / (3 * D), w = (i / D) % 3, c = i % D;
-                d[(t * 3 + w) * DP + c] = __ldcg((w == 2 ? wk.g + ((size_t)(t0 + t) * H + h) * D
-                                                         : (w ? wk.q : wk.k) + ((size_t)(t0 + t) * a.kv_heads + kh) * D) + c);
-            }
+            if (lane < NC && c0 + lane < V)
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(s_v + (stg * TC + t) * NC + lane)),
+                             "l"(a.qkv + (size_t)(t0 + t) * C + voff + c0 + lane) : "memory");
+            if (lane < 2)
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(s_bk + (stg * TC + t) * 2 + lane)),
+                             "l"(wk.bk + ((size_t)(t0 + t) * H + h) * 2 + lane) : "memory");
         }
-        for (uint32_t i = tid; i < nt * NC; i += 256) {
-            const uint32_t t = i / NC, c = i % NC;
-            const float* src = a.qkv + (size_t)(t0 + t) * C + voff + c0 + c;
-            float* dst = s_v + (stg * TC + t) * NC + c;
-            if (c0 + c < V) asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
-        }
-        for (uint32_t i = tid; i < nt * 2; i += 256)
-            asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(s_bk + stg * TC * 2 + i)),
-                         "l"(wk.bk + ((size_t)(t0 + i / 2) * H + h) * 2 + (i & 1)) : "memory");
         cp_commit();
     };
     fetch(0, 0);
+    const bool kind = l & 8, odd = l & 4;             // this lane ends up with S^T k (0) or S^T q (1) of column `odd`
     for (uint32_t t0 = 0, stg = 0; t0 < rows; t0 += TC, stg ^= 1) {
         fetch(t0 + TC, stg ^ 1);
         cp_wait<1>();
         __syncthreads();
         const uint32_t nt = min(TC, rows - t0);
         const float* kqg = s_kqg + stg * TC * 3 * DP + l * 4;
-#pragma unroll 2
-        for (uint32_t t = 0; t < nt; t++) {
+        uint64_t k[RPL / 2], q[RPL / 2], gd[RPL / 2];
+        auto load = [&](uint32_t t) {
             const float* p = kqg + t * 3 * DP;
-            float k[RPL], sk[4] = {0.f, 0.f, 0.f, 0.f}, sq[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < RPL; i += 4) {
-                const float4 k4 = *(const float4*)(p + i * LPC), q4 = *(const float4*)(p + DP + i * LPC), g4 = *(const float4*)(p + 2 * DP + i * LPC);
-                k[i] = k4.x; k[i + 1] = k4.y; k[i + 2] = k4.z; k[i + 3] = k4.w;
-                S[i] *= g4.x; S[i + 1] *= g4.y; S[i + 2] *= g4.z; S[i + 3] *= g4.w;
-                sk[0] = fmaf(S[i], k4.x, sk[0]); sk[1] = fmaf(S[i + 1], k4.y, sk[1]); sk[2] = fmaf(S[i + 2], k4.z, sk[2]); sk[3] = fmaf(S[i + 3], k4.w, sk[3]);
-                sq[0] = fmaf(S[i], q4.x, sq[0]); sq[1] = fmaf(S[i + 1], q4.y, sq[1]); sq[2] = fmaf(S[i + 2], q4.z, sq[2]); sq[3] = fmaf(S[i + 3], q4.w, sq[3]);
+                const ulonglong2 k2 = *(const ulonglong2*)(p + i * 16), q2 = *(const ulonglong2*)(p + DP + i * 16), g2 = *(const ulonglong2*)(p + 2 * DP + i * 16);
+                k[i / 2] = k2.x; k[i / 2 + 1] = k2.y;
+                q[i / 2] = q2.x; q[i / 2 + 1] = q2.y;
+                gd[i / 2] = g2.x; gd[i / 2 + 1] = g2.y;
             }
-            float ak = (sk[0] + sk[1]) + (sk[2] + sk[3]), aq = (sq[0] + sq[1]) + (sq[2] + sq[3]);
-#pragma unroll
-            for (int o = 1; o < LPC; o <<= 1) {
-                ak += __shfl_xor_sync(0xffffffffu, ak, o);
-                aq += __shfl_xor_sync(0xffffffffu, aq, o);
-            }
+        };
+        load(0);
+        for (uint32_t t = 0; t < nt; t++) {
             const float2 bk = *(const float2*)(s_bk + (stg * TC + t) * 2);
-            const float u = bk.x * (s_v[(stg * TC + t) * NC + warp * CPW + lane / LPC] - ak);
-            if (l == 0 && col < V) a.o[((size_t)(t0 + t) * H + h) * V + col] = fmaf(u, bk.y, aq);
+            const float vm = s_v[(stg * TC + t) * NC + cl + odd];
+            uint64_t kc[RPL / 2], ak[2], aq[2];
 #pragma unroll
-            for (int i = 0; i < RPL; i++) S[i] = fmaf(k[i], u, S[i]);
+            for (int i = 0; i < RPL / 2; i++) {
+                kc[i] = k[i];
+#pragma unroll
+                for (int c = 0; c < 2; c++) {
+                    S[i][c] = mul2(S[i][c], gd[i]);
+                    ak[c] = i == 0 ? mul2(S[0][c], k[0]) : fma2(S[i][c], k[i], ak[c]);
+                    aq[c] = i == 0 ? mul2(S[0][c], q[0]) : fma2(S[i][c], q[i], aq[c]);
+                }
+            }
+            if (t + 1 < nt) load(t + 1);
+            const float k0 = sum2(ak[0]), k1 = sum2(ak[1]), q0 = sum2(aq[0]), q1 = sum2(aq[1]);
+            const float e0 = (kind ? q0 : k0) + __shfl_xor_sync(0xffffffffu, kind ? k0 : q0, 8);
+            const float e1 = (kind ? q1 : k1) + __shfl_xor_sync(0xffffffffu, kind ? k1 : q1, 8);
+            float e = (odd ? e1 : e0) + __shfl_xor_sync(0xffffffffu, odd ? e0 : e1, 4);
+            e += __shfl_xor_sync(0xffffffffu, e, 2);
+            e += __shfl_xor_sync(0xffffffffu, e, 1);
+            const float um = bk.x * (vm - e);         // u of column `odd`, in the lanes of kind 0
+            const float u0 = __shfl_sync(0xffffffffu, um, base), u1 = __shfl_sync(0xffffffffu, um, base | 4);
+            const uint64_t uu0 = pk2(u0, u0), uu1 = pk2(u1, u1);
+#pragma unroll
+            for (int i = 0; i < RPL / 2; i++) {
+                S[i][0] = fma2(kc[i], uu0, S[i][0]);
+                S[i][1] = fma2(kc[i], uu1, S[i][1]);
+            }
+            if (kind && !(l & 3) && c0 + cl + odd < V) a.o[((size_t)(t0 + t) * H + h) * V + c0 + cl + odd] = fmaf(odd ? u1 : u0, bk.y, e);
         }
         __syncthreads();
     }
     cp_wait<0>();
 #pragma unroll
-    for (int i = 0; i < RPL; i++) {
+    for (int i = 0; i < RPL; i += 2) {
         const uint32_t r = row_of(i);
-        if (r < D && col < V) Sg[(size_t)r * V + col] = S[i];
+#pragma unroll
+        for (int c = 0; c < 2; c++) {
+            const uint32_t col = c0 + cl + c;
+            if (col >= V) continue;
+            float lo, hi;
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(S[i / 2][c]));
+            if (r < D) Sg[(size_t)r * V + col] = lo;
+            if (r + 1 < D) Sg[(size_t)(r + 1) * V + col] = hi;
+        }
     }
 }
 
@@ -224,20 +265,254 @@ gated_norm_kernel(const float* o, const float* __restrict__ w, const float* gate
     for (uint32_t c = lane; c < V; c += 32) A::st(out + off + c, __ldcg(o + off + c) * inv * __ldg(w + c) * sigmoid_f(__ldcg(gate + off + c)));
 }
 
-template <int LPC, int RPL>
-void launch_scan(cudaStream_t st, const DeltaArgs& a, const DeltaWork& w, uint32_t rows) {
-    constexpr uint32_t DP = LPC * RPL, NC = 8 * (32 / LPC);
-    const size_t smem = (size_t)2 * TC * (3 * DP + NC + 2) * 4;
-    const dim3 grid((a.vdim + NC - 1) / NC, a.heads);
-    static int have_v[64] = {}, have_s[64] = {};
-    if (a.dim % 4 == 0) {
-        ensure_dyn_smem(delta_scan_kernel<LPC, RPL, true>, smem, have_v);
-        launch_pdl(delta_scan_kernel<LPC, RPL, true>, grid, dim3(256), smem, st, a, w, rows);
-    } else {
-        ensure_dyn_smem(delta_scan_kernel<LPC, RPL, false>, smem, have_s);
-        launch_pdl(delta_scan_kernel<LPC, RPL, false>, grid, dim3(256), smem, st, a, w, rows);
+// A cluster of ceil(V / 32) CTAs per head, 32 value columns each: convolution of the head's q, k and its values, unit
+// norms, decays and gates from the low-rank vectors, the recurrence, and the gated norm (sum of squares over the cluster).
+// Thread (l = warp, c = lane) holds rows l * RPL .. + RPL - 1 of column c of S. What no earlier kernel of the run writes
+// (S, the window, weights) is requested before the dependency wait. R: rows of the run, 1 or up to 4.
+constexpr uint32_t STEP_ROWS = 4, STEP_COLS = 32;
+inline uint32_t step_floats(const DeltaArgs& a, uint32_t dp, uint32_t r) { return r * (3 * dp + ((a.rank_a + 3) & ~3u) + ((a.rank_g + 3) & ~3u)) + 8 * STEP_COLS * 2; }
+
+// elements k .. k + 3 of row `row` of w [.., n], zeros past n
+__device__ __forceinline__ float4 low_rank4(const uint16_t* __restrict__ w, size_t row, uint32_t k, uint32_t n) {
+    const uint16_t* p = w + row * n + k;
+    if ((n & 3u) == 0) {
+        if (k >= n) return make_float4(0.f, 0.f, 0.f, 0.f);
+        const uint2 q = __ldg((const uint2*)p);
+        return make_float4(bf2f((uint16_t)(q.x & 0xffffu)), bf2f((uint16_t)(q.x >> 16)), bf2f((uint16_t)(q.y & 0xffffu)), bf2f((uint16_t)(q.y >> 16)));
     }
+    return make_float4(k < n ? bf2f(__ldg(p)) : 0.f, k + 1 < n ? bf2f(__ldg(p + 1)) : 0.f, k + 2 < n ? bf2f(__ldg(p + 2)) : 0.f, k + 3 < n ? bf2f(__ldg(p + 3)) : 0.f);
+}
+
+template <class A, int RPL, int R>
+__global__ void __launch_bounds__(256, 1)
+delta_step_kernel(const DeltaArgs a, uint32_t rows_arg) {
+    constexpr uint32_t DP = 8 * RPL, NI = (2 * DP + STEP_COLS + 255) / 256;
+    const uint32_t rows = R == 1 ? 1 : rows_arg;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float s_v[R][STEP_COLS], s_gate[R][STEP_COLS], s_o[R][STEP_COLS], s_n[R][4], s_ss[8][R];
+    cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
+    const uint32_t D = a.dim, V = a.vdim, H = a.heads, KH = a.kv_heads, C = a.channels(), ra4 = (a.rank_a + 3) & ~3u, rg4 = (a.rank_g + 3) & ~3u;
+    float *s_k = sm, *s_q = s_k + R * DP, *s_g = s_q + R * DP;        // [R][DP], zero past D
+    float *s_a1 = s_g + R * DP, *s_g1 = s_a1 + R * ra4;               // [R][rank rounded up to 4], zero past the rank
+    float2* s_part = (float2*)(s_g1 + R * rg4);                       // [8][32]
+    cluster_arrive();
+    pdl_release();
+    const uint32_t tid = threadIdx.x, c = tid & 31, l = tid >> 5, h = blockIdx.y, kh = h / (H / KH), c0 = blockIdx.x * STEP_COLS, col = c0 + c;
+    const int keep = (int)a.taps - 1;
+    const bool four_taps = a.taps == 4;
+    const uint32_t par = *(volatile const uint32_t*)a.conv_count & 1u;      // moves at the end of a run only
+    const float* bank = a.conv_state + (size_t)par * keep * C;
+    float* next = a.conv_state + (size_t)(par ^ 1u) * keep * C;
+    // ---- before the wait
+    float* Sg = a.S + (size_t)h * D * V;
+    float S[RPL];
+#pragma unroll
+    for (int i = 0; i < RPL; i++) {
+        const uint32_t r = l * RPL + i;
+        S[i] = (r < D && col < V) ? __ldcg(Sg + (size_t)r * V + col) : 0.0f;
+    }
+    // channel of convolution item tid + 256 i: q [DP], k [DP], values [32]; C = none
+    uint32_t ch[NI];
+    float4 cw[NI];
+    float win[NI][3];
+#pragma unroll
+    for (int i = 0; i < (int)NI; i++) {
+        const uint32_t it = tid + 256 * i;
+        ch[i] = it < DP ? (it < D ? kh * D + it : C)
+              : it < 2 * DP ? (it - DP < D ? (KH + kh) * D + it - DP : C)
+              : it < 2 * DP + STEP_COLS && c0 + it - 2 * DP < V ? 2 * KH * D + h * V + c0 + it - 2 * DP : C;
+        if (four_taps && ch[i] < C) {
+            cw[i] = __ldg((const float4*)a.conv_w + ch[i]);
+#pragma unroll
+            for (int j = 0; j < 3; j++) win[i][j] = __ldcg(bank + (size_t)j * C + ch[i]);
+        }
+    }
+    constexpr int PRE = RPL < 16 ? RPL : 16;
+    float4 wa[PRE], wg[STEP_COLS / 8];
+#pragma unroll
+    for (int i = 0; i < PRE; i++) wa[i] = l + 8 * i < D ? low_rank4(a.a2, h * D + l + 8 * i, c * 4, a.rank_a) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < (int)STEP_COLS / 8; j++)
+        wg[j] = c0 + l + 8 * j < V ? low_rank4(a.g2, h * V + c0 + l + 8 * j, c * 4, a.rank_g) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float ea = expf(__ldg(a.a_log + h)), dtb = tid < D ? __ldg(a.dt_bias + h * D + tid) : 0.0f, nw = col < V ? __ldg(a.norm_w + col) : 0.0f;
+    pdl_wait();
+    // ---- the joined projection's rows
+    const typename A::T* y = (const typename A::T*)a.y;
+    const bool qk_keeper = blockIdx.x == 0 && h % (H / KH) == 0;      // one CTA per key head writes the window of q and k
+#pragma unroll
+    for (int i = 0; i < (int)NI; i++) {
+        const uint32_t it = tid + 256 * i;
+        if (it >= 2 * DP + STEP_COLS) break;
+        float* out = it < DP ? s_q + it : it < 2 * DP ? s_k + it - DP : &s_v[0][it - 2 * DP];
+        const uint32_t stride = it < 2 * DP ? DP : STEP_COLS;
+        if (ch[i] >= C) {
+            for (uint32_t r = 0; r < rows; r++) out[r * stride] = 0.0f;
+            continue;
+        }
+        const bool keeper = it >= 2 * DP || qk_keeper;
+        if (four_taps) {
+            float x0 = win[i][0], x1 = win[i][1], x2 = win[i][2];
+#pragma unroll
+            for (int r = 0; r < R; r++) {
+                if (R > 1 && r >= (int)rows) break;
+                const float x3 = A::ld(y + (size_t)r * a.ys + ch[i]);
+                out[r * stride] = silu_f(fmaf(cw[i].w, x3, fmaf(cw[i].z, x2, fmaf(cw[i].y, x1, cw[i].x * x0))));
+                x0 = x1; x1 = x2; x2 = x3;
+            }
+            if (keeper) { next[ch[i]] = x0; next[(size_t)C + ch[i]] = x1; next[2 * (size_t)C + ch[i]] = x2; }
+        } else {
+            for (uint32_t r = 0; r < rows; r++) {
+                float s = 0.0f;
+                for (int j = 0; j < (int)a.taps; j++)
+                    s = fmaf(__ldg(a.conv_w + (size_t)ch[i] * a.taps + j), conv_in<A>(y, bank, (int)r - keep + j, ch[i], a.ys, C, keep), s);
+                out[r * stride] = silu_f(s);
+            }
+            if (keeper)
+                for (int j = 0; j < keep; j++) next[(size_t)j * C + ch[i]] = conv_in<A>(y, bank, (int)rows - keep + j, ch[i], a.ys, C, keep);
+        }
+    }
+    for (uint32_t i = tid; i < rows * (ra4 + rg4); i += 256) {
+        const uint32_t r = i / (ra4 + rg4), k = i % (ra4 + rg4);
+        const typename A::T* yr = y + (size_t)r * a.ys;
+        if (k < ra4) s_a1[r * ra4 + k] = k < a.rank_a ? A::ld(yr + a.a_col + k) : 0.0f;
+        else s_g1[r * rg4 + k - ra4] = k - ra4 < a.rank_g ? A::ld(yr + a.g_col + k - ra4) : 0.0f;
+    }
+    const float blog = l < rows ? A::ld(y + (size_t)l * a.ys + a.b_col + h) : 0.0f;
+    __syncthreads();
+    // ---- norms (warp r: row r), decays and gates (a warp per output)
+    if (l < rows) {
+        float qq = 0.0f, kk = 0.0f, qk = 0.0f;
+        for (uint32_t i = c; i < D; i += 32) {
+            const float qv = s_q[l * DP + i], kv = s_k[l * DP + i];
+            qq = fmaf(qv, qv, qq); kk = fmaf(kv, kv, kk); qk = fmaf(qv, kv, qk);
+        }
+        qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+        if (c == 0) {
+            const float iq = 1.0f / sqrtf((float)D) / sqrtf(qq + 1e-6f), ik = 1.0f / sqrtf(kk + 1e-6f);
+            s_n[l][0] = iq; s_n[l][1] = ik; s_n[l][2] = qk * iq * ik; s_n[l][3] = sigmoid_f(blog);
+        }
+    }
+    auto dot4 = [&](float4 w, const float* x, uint32_t k, uint32_t n4) -> float {
+        if (k >= n4) return 0.0f;
+        const float4 v = *(const float4*)(x + k);
+        return fmaf(w.w, v.w, fmaf(w.z, v.z, fmaf(w.y, v.y, w.x * v.x)));
+    };
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+        if (R > 1 && r >= (int)rows) break;
+        float da[RPL], dg[STEP_COLS / 8];
+#pragma unroll
+        for (int i = 0; i < RPL; i++) {
+            const uint32_t d = l + 8 * i;
+            da[i] = 0.0f;
+            if (d >= D) continue;
+            da[i] = dot4(i < PRE ? wa[i < PRE ? i : 0] : low_rank4(a.a2, h * D + d, c * 4, a.rank_a), s_a1 + r * ra4, c * 4, ra4);
+            for (uint32_t k = 128 + c * 4; k < ra4; k += 128) da[i] += dot4(low_rank4(a.a2, h * D + d, k, a.rank_a), s_a1 + r * ra4, k, ra4);
+        }
+#pragma unroll
+        for (int j = 0; j < (int)STEP_COLS / 8; j++) {
+            const uint32_t v = c0 + l + 8 * j;
+            dg[j] = 0.0f;
+            if (v >= V) continue;
+            dg[j] = dot4(wg[j], s_g1 + r * rg4, c * 4, rg4);
+            for (uint32_t k = 128 + c * 4; k < rg4; k += 128) dg[j] += dot4(low_rank4(a.g2, h * V + v, k, a.rank_g), s_g1 + r * rg4, k, rg4);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+#pragma unroll
+            for (int i = 0; i < RPL; i++) da[i] += __shfl_xor_sync(0xffffffffu, da[i], o);
+#pragma unroll
+            for (int j = 0; j < (int)STEP_COLS / 8; j++) dg[j] += __shfl_xor_sync(0xffffffffu, dg[j], o);
+        }
+#pragma unroll
+        for (int i = 0; i < RPL; i++) if (c == (i & 31)) s_g[r * DP + l + 8 * i] = da[i];
+#pragma unroll
+        for (int j = 0; j < (int)STEP_COLS / 8; j++) if (c == j) s_gate[r][l + 8 * j] = dg[j];
+    }
+    __syncthreads();
+    for (uint32_t r = 0; r < rows; r++)
+        if (tid < DP) {
+            const uint32_t i = r * DP + tid;
+            s_g[i] = tid < D ? expf(-ea * softplus_f(s_g[i] + dtb)) : 0.0f;
+            s_q[i] *= s_n[r][0];
+            s_k[i] *= s_n[r][1];
+        }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+        if (R > 1 && r >= (int)rows) break;
+        float ak = 0.0f, aq = 0.0f, kreg[RPL];
+#pragma unroll
+        for (int i = 0; i < RPL; i += 4) {
+            const float4 g4 = *(const float4*)(s_g + r * DP + l * RPL + i), k4 = *(const float4*)(s_k + r * DP + l * RPL + i), q4 = *(const float4*)(s_q + r * DP + l * RPL + i);
+            kreg[i] = k4.x; kreg[i + 1] = k4.y; kreg[i + 2] = k4.z; kreg[i + 3] = k4.w;
+            S[i] *= g4.x; S[i + 1] *= g4.y; S[i + 2] *= g4.z; S[i + 3] *= g4.w;
+            ak = fmaf(S[i], k4.x, ak); ak = fmaf(S[i + 1], k4.y, ak); ak = fmaf(S[i + 2], k4.z, ak); ak = fmaf(S[i + 3], k4.w, ak);
+            aq = fmaf(S[i], q4.x, aq); aq = fmaf(S[i + 1], q4.y, aq); aq = fmaf(S[i + 2], q4.z, aq); aq = fmaf(S[i + 3], q4.w, aq);
+        }
+        s_part[l * 32 + c] = make_float2(ak, aq);
+        __syncthreads();
+        ak = aq = 0.0f;
+#pragma unroll
+        for (int w = 0; w < 8; w++) { const float2 p = s_part[w * 32 + c]; ak += p.x; aq += p.y; }
+        const float u = s_n[r][3] * (s_v[r][c] - ak);
+#pragma unroll
+        for (int i = 0; i < RPL; i++) S[i] = fmaf(kreg[i], u, S[i]);
+        if (l == 0) s_o[r][c] = fmaf(u, s_n[r][2], aq);
+        __syncthreads();
+    }
+    cluster_wait();                                   // every CTA of the cluster has started
+    if (l < rows) {
+        const float o = col < V ? s_o[l][c] : 0.0f, ss = warp_sum(o * o);
+        if (c < gridDim.x) *cl.map_shared_rank(&s_ss[blockIdx.x][l], c) = ss;
+    }
+    cluster_arrive();
+#pragma unroll
+    for (int i = 0; i < RPL; i++) {
+        const uint32_t r = l * RPL + i;
+        if (r < D && col < V) Sg[(size_t)r * V + col] = S[i];
+    }
+    cluster_wait();
+    if (l < rows && col < V) {
+        float ss = 0.0f;
+        for (uint32_t k = 0; k < gridDim.x; k++) ss += s_ss[k][l];
+        const float inv = 1.0f / sqrtf(ss / (float)V + a.eps);
+        A::st((typename A::T*)a.out + ((size_t)l * H + h) * V + col, s_o[l][c] * inv * nw * sigmoid_f(s_gate[l][c]));
+    }
+}
+
+template <class A, int RPL, int R>
+bool launch_step_r(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
+    static int have[64] = {};
+    const uint32_t vs = (a.vdim + STEP_COLS - 1) / STEP_COLS;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(vs, a.heads); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = (size_t)step_floats(a, 8 * RPL, R) * 4; cfg.stream = st;
+    if (cfg.dynamicSmemBytes > 100 * 1024 || !ensure_dyn_smem(delta_step_kernel<A, RPL, R>, cfg.dynamicSmemBytes, have)) return false;
+    if (launch_pdl_cluster(delta_step_kernel<A, RPL, R>, cfg, dim3(vs, 1, 1), a, rows) != cudaSuccess) { cudaGetLastError(); return false; }
     g_launches++;
+    return true;
+}
+template <class A, int RPL>
+bool launch_step(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
+    return rows == 1 ? launch_step_r<A, RPL, 1>(st, a, rows) : launch_step_r<A, RPL, (int)STEP_ROWS>(st, a, rows);
+}
+
+// Ordinary launch: CTAs that come up while the kernel before still holds SMs pile up on the ones it has left, and the
+// recurrence then runs at the pace of the fullest SM.
+template <int RPL, int NW, bool VEC>
+void launch_scan_t(cudaStream_t st, const DeltaArgs& a, const DeltaWork& w, uint32_t rows) {
+    const size_t smem = (size_t)2 * TC * (3 * 16 * RPL + NW * 4 + 2) * 4;
+    static int have[64] = {};
+    ensure_dyn_smem(delta_scan_kernel<RPL, NW, VEC>, smem, have);
+    delta_scan_kernel<RPL, NW, VEC><<<dim3((a.vdim + NW * 4 - 1) / (NW * 4), a.heads), NW * 32, smem, st>>>(a, w, rows);
+    g_launches++;
+}
+template <int RPL>
+void launch_scan(cudaStream_t st, const DeltaArgs& a, const DeltaWork& w, uint32_t rows) {
+    if (a.dim % 4) { launch_scan_t<RPL, 8, false>(st, a, w, rows); return; }
+    // narrower CTAs while those of 8 warps would leave half of the SMs without one
+    if ((a.vdim + 31) / 32 * a.heads <= 74) launch_scan_t<RPL, 4, true>(st, a, w, rows);
+    else launch_scan_t<RPL, 8, true>(st, a, w, rows);
 }
 
 }  // namespace
@@ -261,11 +536,16 @@ void k_channel_delta(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
     if (a.bf16) launch_pdl(delta_prep_kernel<ActBf16>, dim3(rows), dim3(256), (size_t)a.kv_heads * 4, st, a, w);
     else launch_pdl(delta_prep_kernel<ActF32>, dim3(rows), dim3(256), (size_t)a.kv_heads * 4, st, a, w);
     g_launches++;
-    if (a.dim <= 32) launch_scan<8, 4>(st, a, w, rows);
-    else if (a.dim <= 64) launch_scan<8, 8>(st, a, w, rows);
-    else if (a.dim <= 128) launch_scan<8, 16>(st, a, w, rows);
-    else if (a.dim <= 256) launch_scan<16, 16>(st, a, w, rows);
-    else launch_scan<32, 16>(st, a, w, rows);
+    if (a.dim <= 64) launch_scan<4>(st, a, w, rows);
+    else if (a.dim <= 128) launch_scan<8>(st, a, w, rows);
+    else if (a.dim <= 256) launch_scan<16>(st, a, w, rows);
+    else launch_scan<32>(st, a, w, rows);
+}
+
+bool k_delta_step(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
+    if (!rows || rows > STEP_ROWS || a.dim > 256 || a.vdim > 8 * STEP_COLS) return false;
+    if (a.bf16) return a.dim <= 64 ? launch_step<ActBf16, 8>(st, a, rows) : a.dim <= 128 ? launch_step<ActBf16, 16>(st, a, rows) : launch_step<ActBf16, 32>(st, a, rows);
+    return a.dim <= 64 ? launch_step<ActF32, 8>(st, a, rows) : a.dim <= 128 ? launch_step<ActF32, 16>(st, a, rows) : launch_step<ActF32, 32>(st, a, rows);
 }
 
 void k_gated_norm(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {

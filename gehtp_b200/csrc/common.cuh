@@ -64,15 +64,31 @@ inline bool ensure_dyn_smem(K kernel, size_t bytes, int (&have)[64]) {
 // its predecessor in the stream is still running; the kernel orders itself
 // after the predecessor with griddepcontrol.wait before it touches anything the
 // predecessor wrote (and writes nothing before that point).
+// $GEHTP_CUDA_PDL=0 makes every launch wait for the whole previous kernel (for bisecting ordering faults)
+inline int pdl_allowed() {
+    static const int pdl = [] { const char* e = std::getenv("GEHTP_CUDA_PDL"); return e ? std::atoi(e) : 1; }();
+    return pdl ? 1 : 0;
+}
+
+// The same with thread-block clusters of shape `cl` (grid, block, shared memory and stream in cfg).
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_pdl_cluster(void (*kernel)(KArgs...), cudaLaunchConfig_t cfg, dim3 cl, Args... args) {
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[0].val.programmaticStreamSerializationAllowed = pdl_allowed();
+    at[1].id = cudaLaunchAttributeClusterDimension;
+    at[1].val.clusterDim.x = cl.x; at[1].val.clusterDim.y = cl.y; at[1].val.clusterDim.z = cl.z;
+    cfg.attrs = at; cfg.numAttrs = 2;
+    return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
+}
+
 template <typename... KArgs, typename... Args>
 inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args... args) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = st;
-    // $GEHTP_CUDA_PDL=0 makes every launch wait for the whole previous kernel (for bisecting ordering faults)
-    static const int pdl = [] { const char* e = std::getenv("GEHTP_CUDA_PDL"); return e ? std::atoi(e) : 1; }();
     cudaLaunchAttribute at[1];
     at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    at[0].val.programmaticStreamSerializationAllowed = pdl ? 1 : 0;
+    at[0].val.programmaticStreamSerializationAllowed = pdl_allowed();
     cfg.attrs = at; cfg.numAttrs = 1;
     return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
 }

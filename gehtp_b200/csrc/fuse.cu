@@ -19,6 +19,7 @@
 //                       untransposed tensor through a three-dimensional tensor map
 //   latent attention    LATENT_APPEND + LATENT_ATTEND of a row-count runlist -> for few rows: append and query absorption
 //                       in one kernel, split attention over the cached rows, merge with the value up-projection
+//   delta rule          LINEAR x2 (low-rank decay, gate), SHORT_CONV, CHANNEL_DELTA, GATED_NORM -> for few rows: one kernel
 // and marks the data-movement ops whose result is a constant of the blob (fold_constants).
 //
 // A chain is fused only when every intermediate temp is consumed inside the
@@ -27,6 +28,7 @@
 // (run_range pieces, dump hooks) makes the engine rebuild the plan unfused.
 #include <algorithm>
 #include <cstring>
+#include <functional>
 #include <map>
 #include <utility>
 #include "engine.h"
@@ -138,7 +140,8 @@ struct Span {
                              // 5 prefill split + rotary of q|k|v, 6 swiglu tail behind two GEMMs,
                              // 7 [head][row][d] -> [row][head * d] transposition in front of a W4A16 GEMM,
                              // 8 per-row SLICE + ARGMAX of a matrix joined by a CONCAT tree (greedy sampling of a batch),
-                             // 9 latent append + attention of a row-count runlist
+                             // 9 latent append + attention of a row-count runlist,
+                             // 10 low-rank projections + convolution + delta rule + gated norm of a row-count runlist
     uint32_t first, count;
     std::vector<uint32_t> ops;
     // attention
@@ -535,6 +538,24 @@ bool match_latent_step(const Graph& G, uint32_t i, Span& sp) {
     return true;
 }
 
+// LINEAR (decay) + LINEAR (gate) + SHORT_CONV + CHANNEL_DELTA + GATED_NORM over one joined projection
+bool match_delta_step(const Graph& G, uint32_t i, Span& sp) {
+    const wt_blob* b = G.b;
+    if (i + 4 >= b->n_ops) return false;
+    const wt_op &la = b->ops[i], &lg = b->ops[i + 1], &cv = b->ops[i + 2], &dl = b->ops[i + 3], &gn = b->ops[i + 4];
+    if (la.opcode != OP_LINEAR || lg.opcode != OP_LINEAR || cv.opcode != OP_SHORT_CONV || dl.opcode != OP_CHANNEL_DELTA || gn.opcode != OP_GATED_NORM)
+        return false;
+    const uint32_t y = la.args[0], rows = la.args[3], H = dl.args[9], D = dl.args[11], V = dl.args[12], ys = dl.args[14], bf = dl.args[15] == WT_DT_BF16;
+    if (lg.args[0] != y || cv.args[0] != y || dl.args[2] != y || lg.args[3] != rows || cv.args[4] != rows || dl.args[8] != rows || gn.args[4] != rows) return false;
+    if (dl.args[0] != cv.args[3] || dl.args[1] != la.args[2] || gn.args[0] != dl.args[6] || gn.args[2] != lg.args[2]) return false;
+    if (la.args[5] != H * D || lg.args[5] != H * V || la.args[8] != ys || lg.args[8] != ys || cv.args[7] != ys || gn.args[5] != H || gn.args[6] != V) return false;
+    if (la.args[6] != (bf ? WT_LIN_X_BF16 : 0u) || lg.args[6] != la.args[6] || cv.args[8] != dl.args[15] || gn.args[8] != dl.args[15]) return false;
+    if (cv.args[5] != 2 * dl.args[10] * D + H * V) return false;
+    sp.kind = 10; sp.first = i; sp.count = 5; sp.ops = {i, i + 1, i + 2, i + 3, i + 4};
+    sp.keep = {i, i + 1, i + 2, i + 3};                   // runs of more rows take the ops one after the other
+    return true;
+}
+
 std::vector<Span> g_spans;
 float* g_attn_scratch = nullptr;
 std::map<std::pair<uint32_t, uint64_t>, uint8_t*> g_skip_maps;   // (mask slot, S<<32|Sk) -> device tile-skip bitmap
@@ -606,6 +627,10 @@ void fuse_analyze(const wt_blob* b, const std::vector<PlanOp>& meas, std::vector
     for (uint32_t i = 0; i + 1 < b->n_ops; i++) {
         Span sp{};
         if (!taken[i] && !taken[i + 1] && match_latent_step(G, i, sp)) claim(sp);
+    }
+    for (uint32_t i = 0; i + 4 < b->n_ops; i++) {
+        Span sp{};
+        if (!taken[i] && match_delta_step(G, i, sp)) claim(sp);
     }
     // temps written only by interior ops of chains
     std::vector<int> writes_in(kMaxTemps, 0), writes_out(kMaxTemps, 0);
@@ -687,6 +712,21 @@ void fuse_materialize(const wt_blob* b) {
                 if (k_latent_step(st, l, rows_of(l.rows_arg))) return;
                 append(st);
                 attend(st);
+            };
+        } else if (sp.kind == 10) {
+            std::vector<std::function<void(cudaStream_t)>> parts;
+            for (uint32_t k = 0; k < 5; k++) if (g.plan[sp.first + k].launch) parts.push_back(g.plan[sp.first + k].launch);
+            if (parts.size() != 5) continue;
+            const LinearArgs &la = g.plan[sp.first].rows_args->lin, &lg = g.plan[sp.first + 1].rows_args->lin;
+            DeltaArgs d = g.plan[sp.first + 3].rows_args->del;
+            const DeltaArgs &cv = g.plan[sp.first + 2].rows_args->del, &gn = g.plan[sp.first + 4].rows_args->del;
+            d.conv_w = cv.conv_w; d.conv_state = cv.conv_state; d.conv_count = cv.conv_count; d.taps = cv.taps;
+            d.norm_w = gn.norm_w; d.out = gn.out; d.eps = gn.eps;
+            d.a2 = la.w; d.g2 = lg.w; d.rank_a = la.K; d.rank_g = lg.K;
+            d.a_col = b->ops[sp.first].args[7]; d.g_col = b->ops[sp.first + 1].args[7];
+            head.fused = [=](cudaStream_t st) {
+                if (k_delta_step(st, d, rows_of(d.rows_arg))) return;
+                for (auto& f : parts) f(st);
             };
         } else if (sp.kind == 0) {
             const uint16_t* qkv = (const uint16_t*)resolve(b, sp.qkv);

@@ -7,6 +7,7 @@
 //                          latent_split_kernel (all heads against slices of the cached rows: every row is read once,
 //                          as key and as value), latent_merge_kernel (slices combined, value up-projection, gate)
 //   more bf16 rows         latent_prefill.cu
+#include <cooperative_groups.h>
 #include "launchers_rows.h"
 #include "mma_bf16.cuh"
 
@@ -15,7 +16,7 @@ namespace gehtp {
 namespace {
 
 constexpr uint32_t kAbsorbRows = 16;      // rows up to which the absorbed chain runs
-constexpr uint32_t kSplitCtas = 296;      // target CTAs of the split kernel
+constexpr uint32_t kMaxSplit = 148;       // slices of the cached rows, at most one CTA per SM and query group
 
 // one row's latent, key part and gates, by the whole block: [norm(latent) * w | rotated part | zeros] to the state
 template <class A>
@@ -131,16 +132,18 @@ latent_exact_kernel(const LatentArgs a) {
     }
 }
 
-// Few rows: q of every head into latent space, fp32. Grid (heads + 1, ceil(rank / 64), ceil(rows / 8)); the CTAs of
-// column block 0 add the rotated q part (and the zero tail), the CTAs of x = heads append the latents.
-constexpr int AR = 8;
+// Few rows: q of every head into latent space, times the score scale, stored as hi + lo bf16 rows like the cached ones.
+// Grid (heads + 1, ceil(rank / 64), ceil(rows / AR)), AR = 1 or 8; the CTAs of column block 0 add the rotated q part (and the zero
+// tail), the CTAs of x = heads append the latents.
+constexpr int kAbsorbTile = 8;
+template <int AR>
 __global__ void __launch_bounds__(256)
-latent_absorb_kernel(const LatentArgs a, float* __restrict__ qa, uint32_t rows) {
+latent_absorb_kernel(const LatentArgs a, uint16_t* __restrict__ qh, uint16_t* __restrict__ ql, uint32_t rows) {
     extern __shared__ float sq[];                  // [AR][dim]
     __shared__ float red[8][AR][64 + 2];
     __shared__ float part[8];
     pdl_release();
-    const uint32_t tid = threadIdx.x, h = blockIdx.x, r0 = blockIdx.z * AR, nr = min((uint32_t)AR, rows - r0);
+    const uint32_t tid = threadIdx.x, h = blockIdx.x, r0 = blockIdx.z * AR, nr = AR == 1 ? 1u : min((uint32_t)AR, rows - r0);
     const uint16_t* yb = (const uint16_t*)a.y;
     if (h == a.heads) {
         pdl_wait();
@@ -155,6 +158,12 @@ latent_absorb_kernel(const LatentArgs a, float* __restrict__ qa, uint32_t rows) 
     const uint32_t c = c0 + 2 * cp;
     const uint16_t* w = a.w_kv + (size_t)h * a.dim * a.rank + c;
     const bool pair = (a.rank & 1u) == 0;
+    auto put = [&](size_t i, float v) {
+        v *= a.scale;
+        const uint16_t hi = f2bf(v);
+        qh[i] = hi;
+        ql[i] = f2bf(v - bf2f(hi));
+    };
     // this thread's first weights are requested before the wait
     uint32_t wv[16];
     auto loadw = [&](uint32_t d) -> uint32_t {
@@ -175,13 +184,12 @@ latent_absorb_kernel(const LatentArgs a, float* __restrict__ qa, uint32_t rows) 
             const float2 cs = __ldg((const float2*)a.rope + (size_t)(base + r0 + r) * half + p);
             const uint16_t* s = yb + (size_t)(r0 + r) * yc + h * hd + a.dim + 2 * p;
             const float u = bf2f(__ldcg(s)), v = bf2f(__ldcg(s + 1));
-            float* d = qa + ((size_t)(r0 + r) * a.heads + h) * ls + a.rank + 2 * p;
-            d[0] = u * cs.x - v * cs.y;
-            d[1] = v * cs.x + u * cs.y;
+            put(((size_t)(r0 + r) * a.heads + h) * ls + a.rank + 2 * p, u * cs.x - v * cs.y);
+            put(((size_t)(r0 + r) * a.heads + h) * ls + a.rank + 2 * p + 1, v * cs.x + u * cs.y);
         }
         const uint32_t tail = ls - a.rank - a.rot;
         for (uint32_t i = tid; i < nr * tail; i += 256)
-            qa[((size_t)(r0 + i / tail) * a.heads + h) * ls + a.rank + a.rot + i % tail] = 0.0f;
+            put(((size_t)(r0 + i / tail) * a.heads + h) * ls + a.rank + a.rot + i % tail, 0.0f);
     }
     __syncthreads();
     float acc[AR][2];
@@ -199,7 +207,7 @@ latent_absorb_kernel(const LatentArgs a, float* __restrict__ qa, uint32_t rows) 
             const float w0 = bf2f((uint16_t)(wv[u] & 0xffffu)), w1 = bf2f((uint16_t)(wv[u] >> 16));
 #pragma unroll
             for (int r = 0; r < AR; r++) {
-                if (r >= nr) break;
+                if (AR > 1 && r >= (int)nr) break;
                 const float q = sq[r * a.dim + d];
                 acc[r][0] = fmaf(q, w0, acc[r][0]);
                 acc[r][1] = fmaf(q, w1, acc[r][1]);
@@ -215,7 +223,7 @@ latent_absorb_kernel(const LatentArgs a, float* __restrict__ qa, uint32_t rows) 
         float s = 0.0f;
 #pragma unroll
         for (int j = 0; j < 8; j++) s += red[j][r][k];
-        qa[((size_t)(r0 + r) * a.heads + h) * ls + c0 + k] = s;
+        put(((size_t)(r0 + r) * a.heads + h) * ls + c0 + k, s);
     }
 }
 
@@ -227,7 +235,7 @@ latent_absorb_kernel(const LatentArgs a, float* __restrict__ qa, uint32_t rows) 
 constexpr int TP = 32, STG = 3;
 template <int NT, int QT>
 __global__ void __launch_bounds__(256)
-latent_split_kernel(const LatentArgs a, const float* qa, float* part_o, float* part_ml, uint32_t rows) {
+latent_split_kernel(const LatentArgs a, const uint16_t* qh, const uint16_t* ql, float* part_o, float* part_ml, uint32_t rows) {
     extern __shared__ __align__(16) unsigned char smem[];
     constexpr int M = 16 * QT;
     const uint32_t ls = a.ls(), rs = ls + 8;                          // padded rows: 16-byte chunks of 8 rows fall into different banks
@@ -243,32 +251,38 @@ latent_split_kernel(const LatentArgs a, const float* qa, float* part_o, float* p
     pdl_release();
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t pairs = rows * a.heads, p0 = blockIdx.y * M, nsplit = gridDim.x;
-    pdl_wait();
-    const uint32_t past = *a.counter, n = min(past + rows, a.nslots);
+    // The position counter moves at the end of a run only, and rows below it were written by earlier runs: tiles that
+    // hold none of this run's rows are requested before the dependency wait.
+    const uint32_t past = *(volatile const uint32_t*)a.counter, n = min(past + rows, a.nslots);
     const uint32_t tiles = (n + TP - 1) / TP, per = (tiles + nsplit - 1) / nsplit;
     const uint32_t t0 = min(blockIdx.x * per, tiles), t1 = min(t0 + per, tiles);
     const uint16_t* st = (const uint16_t*)a.state;
     const uint32_t ch = ls / 8;
     auto fetch = [&](uint32_t t) {
-        if (t < t1) {
-            uint16_t* d = sk + (t % STG) * TP * rs;
-            for (uint32_t i = tid; i < TP * ch; i += 256) {
-                const uint32_t r = i / ch, c = i % ch, pos = t * TP + r;
-                cp16(smem_addr(d + r * rs + c * 8), st + (size_t)min(pos, n - 1) * ls + c * 8, pos < n ? 16 : 0);
-            }
+        if (t >= t1) return;
+        uint16_t* d = sk + (t % STG) * TP * rs;
+        for (uint32_t r = warp; r < TP; r += 8) {
+            const uint32_t pos = t * TP + r;
+            const uint16_t* src = st + (size_t)min(pos, n - 1) * ls;
+            for (uint32_t c = lane; c < ch; c += 32) cp16(smem_addr(d + r * rs + c * 8), src + c * 8, pos < n ? 16 : 0);
         }
-        cp_commit();
     };
-    fetch(t0); fetch(t0 + 1);
-    for (uint32_t i = tid; i < M * (ls / 2); i += 256) {
-        const uint32_t r = i / (ls / 2), c = (i % (ls / 2)) * 2;
-        float2 v = make_float2(0.f, 0.f);
-        if (p0 + r < pairs) v = __ldcg((const float2*)(qa + (size_t)(p0 + r) * ls + c));
-        uint32_t hi, lo;
-        split_bf2(v.x * a.scale, v.y * a.scale, hi, lo);
-        *(uint32_t*)(sqh + r * rs + c) = hi;
-        *(uint32_t*)(sql + r * rs + c) = lo;
+    const bool early0 = (t0 + 1) * TP <= past, early1 = (t0 + 2) * TP <= past;
+    if (early0) fetch(t0);
+    if (early1) fetch(t0 + 1);
+    pdl_wait();
+    for (uint32_t r = warp; r < M; r += 8) {
+        const bool live = p0 + r < pairs;
+        const size_t src = (size_t)(live ? p0 + r : 0) * ls;
+        for (uint32_t c = lane; c < ch; c += 32) {
+            cp16(smem_addr(sqh + r * rs + c * 8), qh + src + c * 8, live ? 16 : 0);
+            cp16(smem_addr(sql + r * rs + c * 8), ql + src + c * 8, live ? 16 : 0);
+        }
     }
+    if (!early0) fetch(t0);
+    cp_commit();
+    if (!early1) fetch(t0 + 1);
+    cp_commit();
     if (tid < M) { sm_m[tid] = -INFINITY; sm_l[tid] = 0.0f; }
     float o[QT][NT][4];
 #pragma unroll
@@ -285,22 +299,40 @@ latent_split_kernel(const LatentArgs a, const float* qa, float* part_o, float* p
         cp_wait<1>();
         __syncthreads();                                              // tile t is here; everyone is done with tile t - 1
         fetch(t + 2);
+        cp_commit();
         const uint16_t* kt = sk + (t % STG) * TP * rs;
         {   // scores of (m tile mt, positions 8 nt .. + 7) over k steps [k_lo, k_hi)
-            float acc[4] = {0.f, 0.f, 0.f, 0.f};
-            const uint32_t qh = smem_addr(sqh + (mt * 16 + a_row) * rs + a_col), ql = smem_addr(sql + (mt * 16 + a_row) * rs + a_col);
-            const uint32_t kb = smem_addr(kt + (nt * 8 + (lane & 7)) * rs + ((lane >> 3) & 1) * 8);
-            for (uint32_t ks = k_lo; ks < k_hi; ks++) {
-                uint32_t ah[4], al[4], b0, b1;
-                ldsm4(ah, qh + ks * 32);
-                ldsm4(al, ql + ks * 32);
-                asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(kb + ks * 32) : "memory");
-                mma_bf16(acc, ah, b0, b1);
-                mma_bf16(acc, al, b0, b1);
+            float acc[2][4] = {}, acl[2][4] = {};                     // four independent chains
+            const uint32_t aqh = smem_addr(sqh + (mt * 16 + a_row) * rs + a_col), aql = smem_addr(sql + (mt * 16 + a_row) * rs + a_col);
+            const uint32_t kb = smem_addr(kt + (nt * 8 + (lane & 7)) * rs + (lane >> 3) * 8);
+            uint32_t ks = k_lo;
+#pragma unroll 3
+            for (; ks + 2 <= k_hi; ks += 2) {
+                uint32_t ah[2][4], al[2][4], b[4];
+                ldsm4(b, kb + ks * 32);                               // two k steps of 8 positions
+                ldsm4(ah[0], aqh + ks * 32);
+                ldsm4(al[0], aql + ks * 32);
+                ldsm4(ah[1], aqh + ks * 32 + 32);
+                ldsm4(al[1], aql + ks * 32 + 32);
+                mma_bf16(acc[0], ah[0], b[0], b[1]);
+                mma_bf16(acl[0], al[0], b[0], b[1]);
+                mma_bf16(acc[1], ah[1], b[2], b[3]);
+                mma_bf16(acl[1], al[1], b[2], b[3]);
             }
+            if (ks < k_hi) {
+                uint32_t ah[4], al[4], b0, b1;
+                ldsm4(ah, aqh + ks * 32);
+                ldsm4(al, aql + ks * 32);
+                const uint32_t k1 = smem_addr(kt + (nt * 8 + (lane & 7)) * rs + ((lane >> 3) & 1) * 8) + ks * 32;
+                asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(k1) : "memory");
+                mma_bf16(acc[0], ah, b0, b1);
+                mma_bf16(acl[0], al, b0, b1);
+            }
+#pragma unroll
+            for (int k = 0; k < 4; k++) acc[0][k] = (acc[0][k] + acc[1][k]) + (acl[0][k] + acl[1][k]);
             float* d = ss + kh * M * (TP + 1) + (mt * 16 + g) * (TP + 1) + nt * 8 + 2 * t4;
-            d[0] = acc[0]; d[1] = acc[1];
-            d[8 * (TP + 1)] = acc[2]; d[8 * (TP + 1) + 1] = acc[3];
+            d[0] = acc[0][0]; d[1] = acc[0][1];
+            d[8 * (TP + 1)] = acc[0][2]; d[8 * (TP + 1) + 1] = acc[0][3];
         }
         __syncthreads();
 #pragma unroll
@@ -376,56 +408,77 @@ latent_split_kernel(const LatentArgs a, const float* qa, float* part_o, float* p
     }
 }
 
-// Slices of one (row, head) pair combined, then vdim / gridDim.y of its values. Dynamic shared memory: [nsplit] weights, [rank] latent.
+// Slices of one (row, head) pair combined, value up-projection, gate. A cluster of 8 CTAs per pair: each combines an
+// eighth of the latent columns (a column by 4 threads, a quarter of the slices each), the pieces meet through
+// distributed shared memory, then each CTA computes an eighth of the values.
+constexpr uint32_t MC = 8, MCOLS = 64;
 __global__ void __launch_bounds__(256)
 latent_merge_kernel(const LatentArgs a, const float* part_o, const float* part_ml, uint32_t nsplit) {
-    extern __shared__ float smf[];
-    __shared__ float red[8];
-    float *sw = smf, *ctx = smf + ((nsplit + 3) & ~3u);
+    __shared__ float sw[kMaxSplit], red[8], quarter[4][MCOLS], ctx[MC * MCOLS];
+    cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
+    cluster_arrive();                                  // paired with the wait in front of the first remote store
+    const uint32_t pr = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = pr % a.heads, part = blockIdx.y;
+    // the weights of this CTA's first 8 values (one per warp) are requested before the wait
+    const uint32_t vper = (a.vdim + MC - 1) / MC, v0 = part * vper, v1 = min(v0 + vper, a.vdim);
+    const bool vec = (a.rank & 7u) == 0;
+    auto wrow = [&](uint32_t v) { return a.w_kv + ((size_t)a.heads * a.dim + (size_t)h * a.vdim + v) * a.rank; };
+    uint4 w0[2];
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+        const uint32_t c = lane * 8 + u * 256;
+        w0[u] = vec && v0 + warp < v1 && c < a.rank ? __ldg((const uint4*)(wrow(v0 + warp) + c)) : make_uint4(0, 0, 0, 0);
+    }
     pdl_wait();
     pdl_release();          // after the wait, like the merge of the KV-ring attention
-    const uint32_t pr = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = pr % a.heads;
-    float m = -INFINITY;
-    for (uint32_t s = tid; s < nsplit; s += 256) m = fmaxf(m, __ldcg(part_ml + ((size_t)pr * nsplit + s) * 2));
-    m = warp_max(m);
+    // nsplit <= kMaxSplit: one slice per thread here, at most kMaxSplit / 4 slices of a column per thread below; the
+    // partial latents are requested before the weights are known
+    const float2 ml = tid < nsplit ? __ldcg((const float2*)part_ml + (size_t)pr * nsplit + tid) : make_float2(-INFINITY, 0.0f);
+    const uint32_t cper = (a.rank + MC - 1) / MC, c = part * cper + tid % MCOLS, q = tid / MCOLS;     // cper <= MCOLS
+    const bool live = tid % MCOLS < cper && c < a.rank;
+    const float* po = part_o + (size_t)pr * nsplit * a.rank + c;
+    float v[kMaxSplit / 4];
+#pragma unroll
+    for (int i = 0; i < (int)kMaxSplit / 4; i++) {
+        const uint32_t s = q + 4 * i;
+        v[i] = live && s < nsplit ? __ldcg(po + (size_t)s * a.rank) : 0.0f;
+    }
+    float m = warp_max(ml.x);
     if (lane == 0) red[warp] = m;
     __syncthreads();
 #pragma unroll
     for (int w = 0; w < 8; w++) m = fmaxf(m, red[w]);
-    float l = 0.0f;
-    for (uint32_t s = tid; s < nsplit; s += 256) {
-        const float2 ml = __ldcg((const float2*)part_ml + (size_t)pr * nsplit + s);
-        const float w = ml.y > 0.0f ? expf(ml.x - m) : 0.0f;       // an empty slice has sum 0
-        sw[s] = w;
-        l += w * ml.y;
-    }
-    l = block_sum(l, red);
-    const float* po = part_o + (size_t)pr * nsplit * a.rank;
-    for (uint32_t c = tid; c < a.rank; c += 256) {
+    const float wt = ml.y > 0.0f ? expf(ml.x - m) : 0.0f;          // an empty slice has sum 0 (and a zero latent)
+    if (tid < kMaxSplit) sw[tid] = wt;
+    const float l = block_sum(wt * ml.y, red);
+    {
         float o = 0.0f;
-#pragma unroll 8
-        for (uint32_t s = 0; s < nsplit; s++) {
-            const float w = sw[s];
-            if (w != 0.0f) o = fmaf(w, __ldcg(po + (size_t)s * a.rank + c), o);
+#pragma unroll
+        for (int i = 0; i < (int)kMaxSplit / 4; i++) o = fmaf(sw[q + 4 * i], v[i], o);
+        quarter[q][tid % MCOLS] = o;
+        __syncthreads();
+        cluster_wait();                                // every CTA of the cluster has started
+        if (tid < cper && part * cper + tid < a.rank) {
+            const float sum = (quarter[0][tid] + quarter[1][tid]) + (quarter[2][tid] + quarter[3][tid]);
+            for (uint32_t k = 0; k < MC; k++) *cl.map_shared_rank(ctx + part * cper + tid, k) = sum;
         }
-        ctx[c] = o;
     }
-    __syncthreads();
+    cl.sync();
     const float gt = a.gate[pr] / l;
-    const uint32_t vper = (a.vdim + gridDim.y - 1) / gridDim.y, v0 = blockIdx.y * vper, v1 = min(v0 + vper, a.vdim);
     uint16_t* out = (uint16_t*)a.out + (size_t)pr * a.vdim;
-    const bool vec = (a.rank & 7u) == 0;
     for (uint32_t v = v0 + warp; v < v1; v += 8) {
-        const uint16_t* w = a.w_kv + ((size_t)a.heads * a.dim + (size_t)h * a.vdim + v) * a.rank;
+        const uint16_t* w = wrow(v);
         float s = 0.0f;
         if (vec) {
-            for (uint32_t c = lane * 8; c < a.rank; c += 256) {
-                const uint4 q = __ldg((const uint4*)(w + c));
-                const uint32_t u[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const uint32_t c = lane * 8 + u * 256;
+                if (c >= a.rank) break;
+                const uint4 q = v == v0 + warp ? w0[u] : __ldg((const uint4*)(w + c));
+                const uint32_t x[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
                 for (int k = 0; k < 4; k++) {
-                    s = fmaf(ctx[c + 2 * k], bf2f((uint16_t)(u[k] & 0xffffu)), s);
-                    s = fmaf(ctx[c + 2 * k + 1], bf2f((uint16_t)(u[k] >> 16)), s);
+                    s = fmaf(ctx[c + 2 * k], bf2f((uint16_t)(x[k] & 0xffffu)), s);
+                    s = fmaf(ctx[c + 2 * k + 1], bf2f((uint16_t)(x[k] >> 16)), s);
                 }
             }
         } else {
@@ -451,18 +504,18 @@ bool split_plan(const LatentArgs& a, uint32_t rows, SplitPlan& s) {
     if (split_smem(a.ls(), (int)s.qt) > 220 * 1024) return false;
     s.groups = (pairs + 16 * s.qt - 1) / (16 * s.qt);
     const uint32_t tiles = (a.nslots + TP - 1) / TP;
-    s.nsplit = kSplitCtas / 2 / s.groups;
+    s.nsplit = kMaxSplit / s.groups;
     if (s.nsplit > (tiles + 1) / 2) s.nsplit = (tiles + 1) / 2;
     if (s.nsplit < 1) s.nsplit = 1;
     return true;
 }
 
 template <int NT, int QT>
-bool launch_split(cudaStream_t st, const LatentArgs& a, const float* qa, float* po, float* pml, uint32_t rows, const SplitPlan& s) {
+bool launch_split(cudaStream_t st, const LatentArgs& a, const uint16_t* qh, const uint16_t* ql, float* po, float* pml, uint32_t rows, const SplitPlan& s) {
     static int have[64] = {};
     const size_t smem = split_smem(a.ls(), QT);
     if (!ensure_dyn_smem(latent_split_kernel<NT, QT>, smem, have)) return false;
-    launch_pdl(latent_split_kernel<NT, QT>, dim3(s.nsplit, s.groups), dim3(256), smem, st, a, qa, po, pml, rows);
+    launch_pdl(latent_split_kernel<NT, QT>, dim3(s.nsplit, s.groups), dim3(256), smem, st, a, qh, ql, po, pml, rows);
     g_launches++;
     return true;
 }
@@ -472,7 +525,7 @@ size_t step_floats(const LatentArgs& a, uint32_t rows) {
     SplitPlan s;
     if (!split_plan(a, rows, s)) return 0;
     const size_t pairs = (size_t)rows * a.heads;
-    return ((pairs * a.ls() + 3) & ~(size_t)3) + ((pairs * s.nsplit * a.rank + 3) & ~(size_t)3) + pairs * s.nsplit * 2;
+    return pairs * a.ls() + ((pairs * s.nsplit * a.rank + 3) & ~(size_t)3) + pairs * s.nsplit * 2;
 }
 
 }  // namespace
@@ -513,23 +566,26 @@ bool k_latent_step(cudaStream_t st, const LatentArgs& a, uint32_t rows) {
     SplitPlan s;
     if (!rows || rows > kAbsorbRows || !split_plan(a, rows, s)) return false;
     const size_t pairs = (size_t)rows * a.heads;
-    float* qa = a.work;
-    float* po = qa + ((pairs * a.ls() + 3) & ~(size_t)3);
+    uint16_t *qh = (uint16_t*)a.work, *ql = qh + pairs * a.ls();      // rows of a multiple of 16 elements
+    float* po = a.work + pairs * a.ls();
     float* pml = po + ((pairs * s.nsplit * a.rank + 3) & ~(size_t)3);
-    launch_pdl(latent_absorb_kernel, dim3(a.heads + 1, (a.rank + 63) / 64, (rows + AR - 1) / AR), dim3(256), (size_t)AR * a.dim * 4, st, a, qa, rows);
+    const dim3 ag(a.heads + 1, (a.rank + 63) / 64, rows == 1 ? 1 : (rows + kAbsorbTile - 1) / kAbsorbTile);
+    if (rows == 1) launch_pdl(latent_absorb_kernel<1>, ag, dim3(256), (size_t)a.dim * 4, st, a, qh, ql, rows);
+    else launch_pdl(latent_absorb_kernel<kAbsorbTile>, ag, dim3(256), (size_t)kAbsorbTile * a.dim * 4, st, a, qh, ql, rows);
     g_launches++;
     bool ok;
     switch (s.nt * 10 + s.qt) {
-    case 21: ok = launch_split<2, 1>(st, a, qa, po, pml, rows, s); break;
-    case 22: ok = launch_split<2, 2>(st, a, qa, po, pml, rows, s); break;
-    case 41: ok = launch_split<4, 1>(st, a, qa, po, pml, rows, s); break;
-    case 42: ok = launch_split<4, 2>(st, a, qa, po, pml, rows, s); break;
-    case 81: ok = launch_split<8, 1>(st, a, qa, po, pml, rows, s); break;
-    default: ok = launch_split<8, 2>(st, a, qa, po, pml, rows, s); break;
+    case 21: ok = launch_split<2, 1>(st, a, qh, ql, po, pml, rows, s); break;
+    case 22: ok = launch_split<2, 2>(st, a, qh, ql, po, pml, rows, s); break;
+    case 41: ok = launch_split<4, 1>(st, a, qh, ql, po, pml, rows, s); break;
+    case 42: ok = launch_split<4, 2>(st, a, qh, ql, po, pml, rows, s); break;
+    case 81: ok = launch_split<8, 1>(st, a, qh, ql, po, pml, rows, s); break;
+    default: ok = launch_split<8, 2>(st, a, qh, ql, po, pml, rows, s); break;
     }
     if (!ok) return false;
-    const uint32_t vs = a.vdim >= 32 && pairs * 4 <= 592 ? 4 : 1;
-    launch_pdl(latent_merge_kernel, dim3((uint32_t)pairs, vs), dim3(256), (((size_t)s.nsplit + 3) / 4 * 4 + a.rank) * 4, st, a, (const float*)po, (const float*)pml, s.nsplit);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((uint32_t)pairs, MC); cfg.blockDim = dim3(256); cfg.stream = st;
+    if (launch_pdl_cluster(latent_merge_kernel, cfg, dim3(1, MC, 1), a, (const float*)po, (const float*)pml, s.nsplit) != cudaSuccess) { cudaGetLastError(); return false; }
     g_launches++;
     return true;
 }

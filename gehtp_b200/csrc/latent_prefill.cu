@@ -50,7 +50,7 @@ latent_flash_kernel(const LatentArgs a, const uint16_t* kv, uint32_t rows, uint3
     uint16_t* sv = sk + 2 * BN * rk;                      // [2][BN][rv]
     pdl_release();
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-    const uint32_t h = blockIdx.y, q0 = (gridDim.x - 1 - blockIdx.x) * BM;       // longest rows first
+    const uint32_t h = blockIdx.x, q0 = (gridDim.y - 1 - blockIdx.y) * BM;       // longest rows of all heads first
     // columns no copy writes: padding of a head to 16
     zero_cols(sq, rk, BM, hd, dp);
     zero_cols(sk, rk, 2 * BN, hd, dp);
@@ -88,6 +88,7 @@ latent_flash_kernel(const LatentArgs a, const uint16_t* kv, uint32_t rows, uint3
 #pragma unroll
         for (int i = 0; i < (int)BN / 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
         const uint32_t kaddr = smem_addr(k + ((lane & 7) + (lane >> 4) * 8) * rk + ((lane >> 3) & 1) * 8);
+#pragma unroll 4
         for (uint32_t ks = 0; ks < dp / 16; ks++) {
             uint32_t qa[4];
             ldsm4(qa, qaddr + ks * 32);
@@ -179,7 +180,7 @@ bool launch_flash(cudaStream_t st, const LatentArgs& a, const uint16_t* kv, uint
     static int have[64] = {};
     const size_t smem = flash_smem(a);
     if (!ensure_dyn_smem(latent_flash_kernel<VT, VEC>, smem, have)) return false;
-    launch_pdl(latent_flash_kernel<VT, VEC>, dim3((rows + BM - 1) / BM, a.heads), dim3(256), smem, st, a, kv, rows, past);
+    launch_pdl(latent_flash_kernel<VT, VEC>, dim3(a.heads, (rows + BM - 1) / BM), dim3(256), smem, st, a, kv, rows, past);
     g_launches++;
     return true;
 }

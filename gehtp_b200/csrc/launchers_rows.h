@@ -61,11 +61,15 @@ struct DeltaArgs {
     float* S; float* o; float* work;
     uint32_t heads, kv_heads, dim, vdim, rows_arg;
     const float* norm_w; const float* gate; void* out; float eps; bool bf16;
+    // one-kernel step: second halves of the low-rank decay and gate projections, columns of their first halves in y
+    const uint16_t *a2, *g2; uint32_t rank_a, rank_g, a_col, g_col;
     __host__ __device__ uint32_t channels() const { return 2 * kv_heads * dim + heads * vdim; }
 };
 void k_short_conv(cudaStream_t st, const DeltaArgs& a, uint32_t rows);
 size_t delta_work_floats(const DeltaArgs& a, uint32_t max_rows);
 void k_channel_delta(cudaStream_t st, const DeltaArgs& a, uint32_t rows);
+// all of the above for up to 4 rows in one launch, the low-rank projections included; false: sizes not taken
+bool k_delta_step(cudaStream_t st, const DeltaArgs& a, uint32_t rows);
 void k_gated_norm(cudaStream_t st, const DeltaArgs& a, uint32_t rows);
 
 // what a planned row-count op was resolved to

@@ -26,9 +26,8 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 // An fp32 value as the sum of two bf16 values (about 16 significant bits), pairwise packed: attention weights and
 // absorbed queries enter the tensor cores in this form, two MMAs for one.
 __device__ __forceinline__ void split_bf2(float a, float b, uint32_t& hi, uint32_t& lo) {
-    const uint16_t ha = f2bf(a), hb = f2bf(b);
-    hi = (uint32_t)ha | ((uint32_t)hb << 16);
-    lo = pack_bf2(a - bf2f(ha), b - bf2f(hb));
+    hi = pack_bf2(a, b);
+    lo = pack_bf2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 
 }  // namespace gehtp
