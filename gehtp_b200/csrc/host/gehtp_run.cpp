@@ -12,9 +12,11 @@
 //          first run when it exists, written after the last one, the way the reference's host golden
 //          uses GEHTP_HOST_STATE, compiler/src/ir/graph_prepare.cpp:720,1155). External weights are
 //          looked for beside the blob: <blob minus ".wtop">.weights.bin.
-//   serve: blob, req, resp, out, out_temp, in_bytes; optional idle_exit_s, weights_size, trace.
+//          Row-count runlists: rows, sel (counts of the run).
+//   serve: blob, req, resp, out, out_temp, in_bytes; optional idle_exit_s, weights_size, trace, out_kind
+//          ("token": out_temp holds int32 choices made on the device; else an fp16 face whose arg-max is the token).
 //          A request file is a 4-byte big-endian header length, a JSON header
-//          {"op": "run|reset|ping|shutdown", "want_out": 0|1, ...} and, for run, the input body; it is
+//          {"op": "run|reset|ping|shutdown", "want_out": 0|1, "rows": n, "sel": n} (counts: row-count runlists) and, for run, the input body; it is
 //          unlinked when claimed. The response file is 4-byte big-endian length + JSON
 //          {"rc":0,"token":n,"steps":u,"step_us":u} (token = arg-max of the fp16 output temp).
 // op_ts file: 'WTS1' u32 | version 2 u32 | n_ops u32 | pad u32 | wall_us u64 | n_ops x wt_op_ts.
@@ -132,6 +134,15 @@ bool dump_temp(const std::string& path, uint32_t temp) {
     return n && p && write_file(path, p, n);
 }
 
+// job keys "rows" and "sel": counts of a row-count runlist
+bool set_counts(const wt_blob* b, long rows, long sel) {
+    if (rows <= 0) return true;
+    char err[160] = {0};
+    if (gehtp_cuda_set_rows(b, (uint32_t)rows, (uint32_t)sel, err, sizeof err) == 0) return true;
+    logf("[FAIL] rows %ld sel %ld: %s", rows, sel, err);
+    return false;
+}
+
 int run_step(const wt_blob* b, const std::string& in_path, const std::string& out_path, uint32_t out_temp) {
     std::vector<uint8_t> in;
     char err[160] = {0};
@@ -169,6 +180,7 @@ int mode_job(const std::string& job_path) {
     Loaded L;
     if (!load_blob(job, L)) return 1;
     if (const char* hook = job.get("hook")) { wt_exec_set_hook(hook); logf("[hook] tensor dump spec: %s", hook); }
+    if (!set_counts(L.blob, job.num("rows", 0), job.num("sel", 0))) { wt_exec_shutdown(); return 1; }
     const char* state_p = job.get("state_file");
     if (!state_file_load(L.blob, state_p)) { wt_exec_shutdown(); return 1; }
     const int64_t t_read1 = now_us();
@@ -201,7 +213,7 @@ int mode_job(const std::string& job_path) {
     const int64_t wall = now_us() - t0;
     if (rc) { logf("[FAIL] wt_exec_run_io rc=%d %s", rc, err); wt_exec_shutdown(); return 1; }
     // per-opcode totals, in the runner's log format
-    constexpr int kMaxCode = 64;
+    constexpr int kMaxCode = OP_ROWS_END;
     int64_t tot[kMaxCode] = {0}, mx[kMaxCode] = {0}, sum = 0, top = 0;
     uint32_t cnt[kMaxCode] = {0};
     int top_i = -1;
@@ -312,6 +324,7 @@ int mode_serve(const std::string& job_path) {
     const uint32_t out_temp = (uint32_t)std::strtoul(temp_s, nullptr, 10);
     const size_t in_bytes = (size_t)job.num("in_bytes", 0);
     const long idle_exit_s = job.num("idle_exit_s", 0);
+    const bool token_out = job.get("out_kind") && !std::strcmp(job.get("out_kind"), "token");
     Loaded L;
     if (!load_blob(job, L)) return 1;
     logf("[serve] blob %s out_temp %u in_bytes %zu idle_exit_s %ld", job.get("blob"), out_temp, in_bytes, idle_exit_s);
@@ -351,6 +364,11 @@ int mode_serve(const std::string& job_path) {
             std::memcpy(body.data(), req.data() + 4 + hl, req.size() - 4 - hl);
             char err[160] = {0};
             const int64_t t0 = now_us();
+            const long rows = json_int(hdr, "rows", 0);
+            if (rows > 0 && gehtp_cuda_set_rows(L.blob, (uint32_t)rows, (uint32_t)json_int(hdr, "sel", 1), err, sizeof err) != 0) {
+                write_resp(resp_p, "{\"rc\":-1,\"err\":\"" + json_escape(err) + "\"}");
+                continue;
+            }
             int rc = wt_exec_run_io(L.blob, body.data(), nullptr, out_temp, nullptr, nullptr, err, sizeof err);
             const int64_t us = now_us() - t0;
             char resp[320];
@@ -358,7 +376,11 @@ int mode_serve(const std::string& job_path) {
                 std::snprintf(resp, sizeof resp, "{\"rc\":%d,\"err\":\"%s\"}", rc, json_escape(err).c_str());
                 logf("[run] FAIL rc=%d err=%s", rc, err);
             } else {
-                int tok = argmax_f16(wt_exec_temp(out_temp), wt_exec_temp_last_bytes(out_temp));
+                const uint8_t* out = wt_exec_temp(out_temp);
+                const uint32_t out_n = wt_exec_temp_last_bytes(out_temp);
+                int32_t tok = -1;
+                if (token_out) { if (out && out_n >= 4) std::memcpy(&tok, out + out_n - 4, 4); }   // the last picked row's choice
+                else tok = argmax_f16(out, out_n);
                 if (json_int(hdr, "want_out", 0) && !dump_temp(out_p, out_temp)) logf("[warn] out file not written");
                 steps++;
                 std::snprintf(resp, sizeof resp, "{\"rc\":0,\"token\":%d,\"steps\":%u,\"step_us\":%lld}", tok, steps, (long long)us);

@@ -227,12 +227,13 @@ latent_absorb_kernel(const LatentArgs a, uint16_t* __restrict__ qh, uint16_t* __
     }
 }
 
-// Attention of 16 * QT (row, head) pairs against one slice of the cached rows. Tiles of 32 positions, three in flight.
-//   scores   8 warps over (m tile, 8 positions, half of the latent when QT = 1); q as hi + lo bf16
-//   softmax  a warp per 2 * QT pairs, lane = position; weights to shared memory as hi + lo bf16
+// Attention of 16 * QT (row, head) pairs against one slice of the cached rows. Tiles of 32 positions, two stages.
+//   scores   every warp takes an eighth of the latent for all pairs and positions of the tile, so that each operand
+//            fragment is read from shared memory once; q as hi + lo bf16
+//   softmax  the eight shares added, a warp per 2 * QT pairs, lane = position; weights to shared memory as hi + lo bf16
 //   values   each warp 8 * NT latent columns, accumulators in registers
 // Partial result per pair and slice: latent [rank], maximum, sum.
-constexpr int TP = 32, STG = 3;
+constexpr int TP = 32, STG = 2;
 template <int NT, int QT>
 __global__ void __launch_bounds__(256)
 latent_split_kernel(const LatentArgs a, const uint16_t* qh, const uint16_t* ql, float* part_o, float* part_ml, uint32_t rows) {
@@ -242,8 +243,8 @@ latent_split_kernel(const LatentArgs a, const uint16_t* qh, const uint16_t* ql, 
     uint16_t* sk = (uint16_t*)smem;                                   // [STG][TP][rs]
     uint16_t* sqh = sk + STG * TP * rs;                               // [M][rs] hi, then lo
     uint16_t* sql = sqh + M * rs;
-    float* ss = (float*)(sql + M * rs);                               // [2][M][TP + 1] scores (two halves of the latent)
-    uint16_t* sph = (uint16_t*)(ss + 2 * M * (TP + 1));               // [M][TP + 8] weights hi, then lo
+    float* ss = (float*)(sql + M * rs);                               // [8][M][TP + 1] scores by share of the latent
+    uint16_t* sph = (uint16_t*)(ss + 8 * M * (TP + 1));               // [M][TP + 8] weights hi, then lo
     uint16_t* spl = sph + M * (TP + 8);
     float* sm_m = (float*)(spl + M * (TP + 8));                       // [M] maximum, sum, correction
     float* sm_l = sm_m + M;
@@ -283,6 +284,7 @@ latent_split_kernel(const LatentArgs a, const uint16_t* qh, const uint16_t* ql, 
     cp_commit();
     if (!early1) fetch(t0 + 1);
     cp_commit();
+    cp_wait<1>();
     if (tid < M) { sm_m[tid] = -INFINITY; sm_l[tid] = 0.0f; }
     float o[QT][NT][4];
 #pragma unroll
@@ -292,55 +294,51 @@ latent_split_kernel(const LatentArgs a, const uint16_t* qh, const uint16_t* ql, 
 #pragma unroll
             for (int k = 0; k < 4; k++) o[q][i][k] = 0.0f;
     const uint32_t g = lane >> 2, t4 = lane & 3;
-    const uint32_t mt = QT == 2 ? warp >> 2 : 0, nt = warp & 3, kh = QT == 2 ? 0 : warp >> 2;
-    const uint32_t KS = ls / 16, k_lo = QT == 2 ? 0 : kh * ((KS + 1) / 2), k_hi = QT == 2 ? KS : (kh ? KS : (KS + 1) / 2);
+    const uint32_t KS = ls / 16, k_lo = KS * warp / 8, k_hi = KS * (warp + 1) / 8;      // this warp's k steps
     const uint32_t a_row = lane & 15, a_col = (lane >> 4) * 8;        // ldmatrix addresses of an A tile
     for (uint32_t t = t0; t < t1; t++) {
-        cp_wait<1>();
+        if (t > t0) cp_wait<0>();
         __syncthreads();                                              // tile t is here; everyone is done with tile t - 1
-        fetch(t + 2);
-        cp_commit();
+        if (t > t0) { fetch(t + 1); cp_commit(); }
         const uint16_t* kt = sk + (t % STG) * TP * rs;
-        {   // scores of (m tile mt, positions 8 nt .. + 7) over k steps [k_lo, k_hi)
-            float acc[2][4] = {}, acl[2][4] = {};                     // four independent chains
-            const uint32_t aqh = smem_addr(sqh + (mt * 16 + a_row) * rs + a_col), aql = smem_addr(sql + (mt * 16 + a_row) * rs + a_col);
-            const uint32_t kb = smem_addr(kt + (nt * 8 + (lane & 7)) * rs + (lane >> 3) * 8);
-            uint32_t ks = k_lo;
-#pragma unroll 3
-            for (; ks + 2 <= k_hi; ks += 2) {
-                uint32_t ah[2][4], al[2][4], b[4];
-                ldsm4(b, kb + ks * 32);                               // two k steps of 8 positions
-                ldsm4(ah[0], aqh + ks * 32);
-                ldsm4(al[0], aql + ks * 32);
-                ldsm4(ah[1], aqh + ks * 32 + 32);
-                ldsm4(al[1], aql + ks * 32 + 32);
-                mma_bf16(acc[0], ah[0], b[0], b[1]);
-                mma_bf16(acl[0], al[0], b[0], b[1]);
-                mma_bf16(acc[1], ah[1], b[2], b[3]);
-                mma_bf16(acl[1], al[1], b[2], b[3]);
-            }
-            if (ks < k_hi) {
-                uint32_t ah[4], al[4], b0, b1;
-                ldsm4(ah, aqh + ks * 32);
-                ldsm4(al, aql + ks * 32);
-                const uint32_t k1 = smem_addr(kt + (nt * 8 + (lane & 7)) * rs + ((lane >> 3) & 1) * 8) + ks * 32;
-                asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(k1) : "memory");
-                mma_bf16(acc[0], ah, b0, b1);
-                mma_bf16(acl[0], al, b0, b1);
+        {
+            float acc[QT][TP / 8][4] = {};
+            const uint32_t kb = smem_addr(kt + ((lane & 7) + (lane >> 4) * 8) * rs + ((lane >> 3) & 1) * 8);
+            for (uint32_t ks = k_lo; ks < k_hi; ks++) {
+                uint32_t b[TP / 16][4];
+#pragma unroll
+                for (int j = 0; j < TP / 16; j++) ldsm4(b[j], kb + j * 16 * rs * 2 + ks * 32);        // 16 positions each
+#pragma unroll
+                for (int q = 0; q < QT; q++) {
+                    uint32_t ah[4], al[4];
+                    ldsm4(ah, smem_addr(sqh + (q * 16 + a_row) * rs + a_col) + ks * 32);
+                    ldsm4(al, smem_addr(sql + (q * 16 + a_row) * rs + a_col) + ks * 32);
+#pragma unroll
+                    for (int j = 0; j < TP / 16; j++) {
+                        mma_bf16(acc[q][2 * j], ah, b[j][0], b[j][1]);
+                        mma_bf16(acc[q][2 * j + 1], ah, b[j][2], b[j][3]);
+                        mma_bf16(acc[q][2 * j], al, b[j][0], b[j][1]);
+                        mma_bf16(acc[q][2 * j + 1], al, b[j][2], b[j][3]);
+                    }
+                }
             }
 #pragma unroll
-            for (int k = 0; k < 4; k++) acc[0][k] = (acc[0][k] + acc[1][k]) + (acl[0][k] + acl[1][k]);
-            float* d = ss + kh * M * (TP + 1) + (mt * 16 + g) * (TP + 1) + nt * 8 + 2 * t4;
-            d[0] = acc[0][0]; d[1] = acc[0][1];
-            d[8 * (TP + 1)] = acc[0][2]; d[8 * (TP + 1) + 1] = acc[0][3];
+            for (int q = 0; q < QT; q++)
+#pragma unroll
+                for (int j = 0; j < TP / 8; j++) {
+                    float* d = ss + warp * M * (TP + 1) + (q * 16 + g) * (TP + 1) + j * 8 + 2 * t4;
+                    d[0] = acc[q][j][0]; d[1] = acc[q][j][1];
+                    d[8 * (TP + 1)] = acc[q][j][2]; d[8 * (TP + 1) + 1] = acc[q][j][3];
+                }
         }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < 2 * QT; i++) {
             const uint32_t r = warp * 2 * QT + i, pos = t * TP + lane;
             const uint32_t row = (p0 + r) / a.heads;
-            float s = ss[r * (TP + 1) + lane];
-            if (QT == 1) s += ss[M * (TP + 1) + r * (TP + 1) + lane];
+            float s = 0.0f;
+#pragma unroll
+            for (int w = 0; w < 8; w++) s += ss[w * M * (TP + 1) + r * (TP + 1) + lane];
             if (pos >= n || pos > past + row) s = -INFINITY;
             const float mo = sm_m[r], mn = fmaxf(mo, warp_max(s));
             const float e = mn == -INFINITY ? 0.0f : expf(s - mn);
@@ -491,7 +489,7 @@ latent_merge_kernel(const LatentArgs a, const float* part_o, const float* part_m
 
 size_t split_smem(uint32_t ls, int qt) {
     const size_t M = 16 * qt, rs = ls + 8;
-    return STG * TP * rs * 2 + 2 * M * rs * 2 + 2 * M * (TP + 1) * 4 + 2 * M * (TP + 8) * 2 + 3 * M * 4;
+    return STG * TP * rs * 2 + 2 * M * rs * 2 + 8 * M * (TP + 1) * 4 + 2 * M * (TP + 8) * 2 + 3 * M * 4;
 }
 
 struct SplitPlan { uint32_t nt, qt, groups, nsplit; };

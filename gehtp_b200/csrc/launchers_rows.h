@@ -47,7 +47,7 @@ struct LatentArgs {
 };
 size_t latent_work_floats(const LatentArgs& a, uint32_t max_rows);
 void k_latent_append(cudaStream_t st, const LatentArgs& a, uint32_t rows);
-// n_past: the host's count of positions before this run
+// n_past: the host's count of positions before this run; exact = true launches nothing that depends on it
 void k_latent_attend(cudaStream_t st, const LatentArgs& a, uint32_t rows, uint32_t n_past, bool exact);
 // append + attend for few rows in one chain (rotary, latent, query absorption in one launch); false: not taken
 bool k_latent_step(cudaStream_t st, const LatentArgs& a, uint32_t rows);

@@ -152,8 +152,10 @@ void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p) {
             l.work = (float*)P.temp_get(a[5], latent_work_floats(l, (uint32_t)mr) * 4u, p);
             if (!l.q || !l.gate || !l.w_kv || !l.out || !l.work) FAIL("latent ref fail");
             p.engine = WT_ENG_HMX;
+            // runs that may be captured take the kernel that reads the position count on the device
             if (P.build) p.launch = [=](cudaStream_t st) {
-                k_latent_attend(st, l, rows_of(rows), g.st_count[l.state_idx], !g.opt_fuse || g.exact_ops);
+                const uint32_t n = rows_of(rows);
+                k_latent_attend(st, l, n, g.st_count[l.state_idx], !g.opt_fuse || g.exact_ops || n <= kGraphRows);
             };
         }
         p.rows_args->lat = l;
