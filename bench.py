@@ -888,7 +888,7 @@ def run_design(args, width):
     profiled run with their algorithmic work. Prefill: 2048 tokens from position 0; decode: one token at context 8192."""
     import torch
     import gehtp_b200
-    from gehtp_b200.runlists import DecoderConfig, build_decode_runlist, build_prefill_runlist, decode_face
+    from gehtp_b200.runlists import DecoderConfig, build_decode_runlist, build_gdn_runlist, build_prefill_runlist, decode_face
     from gehtp_b200.session import Session
     from gehtp_b200.wtop import OP, ROWS_AUTO, SEL_AUTO, Engine
     lib = gehtp_b200.lib()
@@ -956,18 +956,15 @@ def run_design(args, width):
                 r = 1 if a[3] == SEL_AUTO else rows
                 k, c = a[4], a[5]
                 yb = 2 if a[6] & 2 else 4
+                if a[7]:     # head of the delta-rule chain: low-rank projections, convolution, recurrence, gated norm
+                    return ("delta rule chain", 2 * H * 128 * 128 * 4 + 2 * 2 * H * 128 * 128 + rows * (4 * H * 128 + 256) * 2,
+                            2.0 * rows * 128 * H * 256)
                 return "linear %dx%d" % (k, c), 2 * k * c + r * (2 * k + yb * c), 2.0 * r * k * c
             if op.opcode in (OP.LATENT_APPEND, OP.LATENT_ATTEND):
                 ctx = past + rows
                 if rows > 16 and op.opcode == OP.LATENT_APPEND:
                     return "latent append + attend", 2 * rows * (H * 192 * 2 + 576), 2.0 * ctx * 512 * H * 256 + 2.0 * H * 320 * rows * (past + rows / 2)
                 return "latent append + attend", ctx * 576 * 2 + H * 256 * 512 * 2, 2.0 * rows * H * (256 * 512 + ctx * 1088)
-            if op.opcode == OP.SHORT_CONV:
-                return "short conv .. gated norm" if rows <= 8 else "short conv", rows * 3 * H * 128 * 6, 0
-            if op.opcode == OP.CHANNEL_DELTA:
-                return "channel delta", rows * H * 128 * 4 * 6 + H * 128 * 128 * 8, 0
-            if op.opcode == OP.GATED_NORM:
-                return "gated norm", rows * H * 128 * 10, 0
             if op.opcode == OP.NORM_RESID:
                 return "norm + residual", n * width * 14, 0
             return "other", 0, 0
@@ -1051,6 +1048,24 @@ def run_design(args, width):
     ms = timed(step, rewind)
     rewind()
     add(cfg.name, "decode ctx %d" % (CTX - 64), ms, 1, units(eng, face, man["token_temp"], work_fixed(1, CTX)))
+    eng.shutdown()
+    # ---- the delta rule of the gated-delta layer (config 5) at the same heads: chunks of 64 tokens, convolution over 3 H 128 channels
+    buf, man = build_gdn_runlist(S_, width, 3 * H * 128, 4, H, 128, 64)
+    eng = Engine(lib, buf)
+    face = np.zeros((S_, width), np.float16)
+    for _ in range(3):
+        eng.run_io(face, man["conv_temp"], None)
+    ms = (ctypes.c_float * eng.blob.n_ops)()
+    assert lib.gehtp_cuda_run_profiled(ctypes.byref(eng.blob), face.ctypes.data, man["conv_temp"], ms, eng.blob.n_ops, err, 256) == 0, err.value
+    total = {}
+    for i in range(eng.blob.n_ops):
+        name = {OP.DELTA_CHUNK: "delta rule, all chunks", OP.CONV1D_SSM: "convolution"}.get(eng.blob.ops[i].opcode)
+        if name:
+            total[name] = total.get(name, 0.0) + ms[i] * 1e3
+    roof = {"delta rule, all chunks": (S_ // 64 * 2 * H * 128 * 128 * 4 + S_ * H * 128 * 8) / hbm / 1e3, "convolution": S_ * 3 * H * 128 * 4 / hbm / 1e3}
+    lines.append({"design": "gated-delta layer (config 5)", "width": width, "heads": H, "phase": "prefill 2048", "ms": sum(total.values()) / 1e3, "tok_s": None,
+                  "units": {n: {"launches": 1, "us": round(u, 2), "roofline_us": round(roof[n], 2), "frac": round(roof[n] / u, 3)} for n, u in total.items()},
+                  "clocks": clocks})
     eng.shutdown()
     return lines
 

@@ -3,14 +3,13 @@
 //   short_conv_kernel    causal depthwise convolution + silu; the last taps - 1 inputs are kept in the state, two banks:
 //                        a run reads the bank of its parity and writes the other, so that no CTA overwrites what
 //                        another still reads
-//   delta_prep_kernel    unit vectors, decays, step sizes, k . q per token, fp32
-//   delta_scan_kernel    the recurrence, token by token: S lives in registers, 2 columns per 16 lanes, both reductions of
-//                        a token (S^T k and S^T q) run side by side; with S' = g S, u = beta (v - S'^T k),
-//                        S = S' + k u^T:  S^T q = S'^T q + u (k . q)
+//   delta_prep_kernel    unit vectors, decays, step sizes and the products of neighbouring tokens' vectors, fp32
+//   delta_scan_kernel    the recurrence, two tokens at a time: S lives in registers, all reductions of both tokens run side
+//                        by side
 //   gated_norm_kernel    RMS norm of a head's read-out, weight, sigmoid gate
 //   delta_step_kernel    all of it for up to 4 rows, with the second halves of the low-rank decay and gate projections
 //
-// The recurrence is the same arithmetic for one token and for a whole prompt, so a cut of the prompt changes nothing.
+// All of it is fp32, token after token: a cut of the prompt changes nothing but roundings.
 #include <cooperative_groups.h>
 #include "launchers_rows.h"
 #include "mma_bf16.cuh"
@@ -65,7 +64,8 @@ short_conv_kernel(const typename A::T* y, const float* __restrict__ w, float* st
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
-// work: k [rows][KH][D], q [rows][KH][D], decay [rows][H][D], {step, k . q} [rows][H][2]
+// work: k [rows][KH][D], q [rows][KH][D], decay [rows][H][D], {step, k . q, (g k') . k, (g k') . q} [rows][H][4] with k' the
+// key of the row before (odd rows only)
 struct DeltaWork { float *k, *q, *g, *bk; };
 __host__ __device__ inline size_t up4(size_t n) { return (n + 3) & ~(size_t)3; }
 inline DeltaWork work_of(const DeltaArgs& a, uint32_t rows) {
@@ -77,40 +77,58 @@ inline DeltaWork work_of(const DeltaArgs& a, uint32_t rows) {
     return w;
 }
 
-template <class A>
+// A warp per head and pair of rows (2 p, 2 p + 1), the head's vectors in registers (DR values per lane).
+template <class A, int DR>
 __global__ void __launch_bounds__(256)
-delta_prep_kernel(const DeltaArgs a, const DeltaWork wk) {
-    extern __shared__ float s_kq[];                   // [kv_heads]
+delta_prep_kernel(const DeltaArgs a, const DeltaWork wk, uint32_t rows) {
     pdl_release();
     pdl_wait();
-    const uint32_t r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = a.dim, KH = a.kv_heads, H = a.heads;
-    const float* x = a.qkv + (size_t)r * a.channels();
-    const float qs = 1.0f / sqrtf((float)D);
-    for (uint32_t h = warp; h < KH; h += 8) {
-        const float *qx = x + h * D, *kx = x + (KH + h) * D;
+    const uint32_t h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = a.dim, KH = a.kv_heads, H = a.heads;
+    if (h >= H) return;
+    const uint32_t rep = H / KH, kh = h / rep, r0 = blockIdx.y * 2;
+    const float qs = 1.0f / sqrtf((float)D), ea = expf(__ldg(a.a_log + h));
+    float kp[DR], k[DR], q[DR], g[DR];
+#pragma unroll
+    for (int j = 0; j < DR; j++) kp[j] = 0.0f;
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+        const uint32_t r = r0 + e;
+        if (r >= rows) break;
+        const float *qx = a.qkv + (size_t)r * a.channels() + kh * D, *kx = qx + KH * D, *ax = a.a + ((size_t)r * H + h) * D;
         float qq = 0.0f, kk = 0.0f, qk = 0.0f;
-        for (uint32_t i = lane; i < D; i += 32) {
-            const float qv = __ldcg(qx + i), kv = __ldcg(kx + i);
-            qq = fmaf(qv, qv, qq); kk = fmaf(kv, kv, kk); qk = fmaf(qv, kv, qk);
+#pragma unroll
+        for (int j = 0; j < DR; j++) {
+            const uint32_t i = lane + 32 * j;
+            const bool in = i < D;
+            q[j] = in ? __ldcg(qx + i) : 0.0f;
+            k[j] = in ? __ldcg(kx + i) : 0.0f;
+            g[j] = in ? __ldcg(ax + i) + __ldg(a.dt_bias + h * D + i) : 0.0f;
+            qq = fmaf(q[j], q[j], qq); kk = fmaf(k[j], k[j], kk); qk = fmaf(q[j], k[j], qk);
         }
         qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
         const float iq = qs / sqrtf(qq + 1e-6f), ik = 1.0f / sqrtf(kk + 1e-6f);
-        for (uint32_t i = lane; i < D; i += 32) {
-            wk.q[((size_t)r * KH + h) * D + i] = __ldcg(qx + i) * iq;
-            wk.k[((size_t)r * KH + h) * D + i] = __ldcg(kx + i) * ik;
+        float m = 0.0f, n = 0.0f;
+#pragma unroll
+        for (int j = 0; j < DR; j++) {
+            const uint32_t i = lane + 32 * j;
+            g[j] = expf(-ea * softplus_f(g[j]));
+            q[j] *= iq; k[j] *= ik;
+            m = fmaf(g[j] * kp[j], k[j], m);
+            n = fmaf(g[j] * kp[j], q[j], n);
+            if (i < D) {
+                wk.g[((size_t)r * H + h) * D + i] = g[j];
+                if (h % rep == 0) {
+                    wk.q[((size_t)r * KH + kh) * D + i] = q[j];
+                    wk.k[((size_t)r * KH + kh) * D + i] = k[j];
+                }
+            }
+            kp[j] = k[j];
         }
-        if (lane == 0) s_kq[h] = qk * iq * ik;
-    }
-    for (uint32_t i = threadIdx.x; i < H * D; i += 256) {
-        const float z = softplus_f(__ldcg(a.a + (size_t)r * H * D + i) + __ldg(a.dt_bias + i));
-        wk.g[(size_t)r * H * D + i] = expf(-expf(__ldg(a.a_log + i / D)) * z);
-    }
-    __syncthreads();
-    const typename A::T* b = (const typename A::T*)a.y + (size_t)r * a.ys + a.b_col;
-    for (uint32_t h = threadIdx.x; h < H; h += 256) {
-        float* d = wk.bk + ((size_t)r * H + h) * 2;
-        d[0] = sigmoid_f(A::ld(b + h));
-        d[1] = s_kq[h / (H / KH)];
+        if (e) { m = warp_sum(m); n = warp_sum(n); }
+        if (lane == 0) {
+            const float b = A::ld((const typename A::T*)a.y + (size_t)r * a.ys + a.b_col + h);
+            *(float4*)(wk.bk + ((size_t)r * H + h) * 4) = make_float4(sigmoid_f(b), qk * iq * ik, m, n);
+        }
     }
 }
 
@@ -120,11 +138,15 @@ __device__ __forceinline__ float sum2(uint64_t v) { float a, b; asm("mov.b64 {%0
 __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
 __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) { uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
 
-// 16 lanes hold 2 neighbouring columns of S, RPL rows each (as RPL / 2 pairs); a warp holds 4 columns, a CTA NW warps of
-// one head. Every value of k, q and g that a lane reads from shared memory serves 2 columns; those of the next token are
-// read while this token's sums are reduced. The four sums of a token (S^T k and S^T q of 2 columns) are reduced over the
-// 16 lanes by halving: an exchange leaves a lane with half of the sums it had, until lane (kind, column, -, -) holds one.
-// Tokens come in chunks of TC through shared memory (cp.async, two stages; VEC = 16-byte copies).
+// 16 lanes hold 2 neighbouring columns of S, RPL rows each (as RPL / 2 pairs of values); a warp holds 4 columns, a CTA NW
+// warps of one head. Tokens are taken two at a time: with P = g1 S, R = g2 P,
+//   u1 = b1 (v1 - P^T k1)                 o1 = P^T q1 + u1 (k1 . q1)
+//   u2 = b2 (v2 - R^T k2 - u1 m)          o2 = R^T q2 + u1 n + u2 (k2 . q2)       m = (g2 k1) . k2, n = (g2 k1) . q2
+//   S  = R + (g2 k1) u1^T + k2 u2^T
+// so that the four sums of both tokens are reduced together. The eight sums of a lane (4 per column) are reduced over its
+// 16 lanes by halving - an exchange leaves a lane with half of the sums it had - until lane (token, k or q, column, -)
+// holds one. Tokens come in chunks of TC through shared memory (cp.async, two stages; VEC = 16-byte copies); a last odd
+// token is paired with one that changes nothing (decay 1, key, query and step 0).
 constexpr uint32_t TC = 16;
 template <int RPL, int NW, bool VEC>
 __global__ void __launch_bounds__(NW * 32)
@@ -133,7 +155,7 @@ delta_scan_kernel(const DeltaArgs a, const DeltaWork wk, uint32_t rows) {
     extern __shared__ __align__(16) float sm[];
     float* s_kqg = sm;                                // [2][TC][3][DP]
     float* s_v = s_kqg + 2 * TC * 3 * DP;             // [2][TC][NC]
-    float* s_bk = s_v + 2 * TC * NC;                  // [2][TC][2]
+    float* s_bk = s_v + 2 * TC * NC;                  // [2][TC][4]
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, H = a.heads, D = a.dim, V = a.vdim;
     const uint32_t h = blockIdx.y, kh = h / (H / a.kv_heads), c0 = blockIdx.x * NC;
     const uint32_t l = lane & 15, base = lane & 16, cl = warp * 4 + (lane >> 4) * 2;      // first of this lane's columns, within the CTA
@@ -175,62 +197,77 @@ delta_scan_kernel(const DeltaArgs a, const DeltaWork wk, uint32_t rows) {
             if (lane < NC && c0 + lane < V)
                 asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(s_v + (stg * TC + t) * NC + lane)),
                              "l"(a.qkv + (size_t)(t0 + t) * C + voff + c0 + lane) : "memory");
-            if (lane < 2)
-                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(s_bk + (stg * TC + t) * 2 + lane)),
-                             "l"(wk.bk + ((size_t)(t0 + t) * H + h) * 2 + lane) : "memory");
+            if (lane == 0) cp16(smem_addr(s_bk + (stg * TC + t) * 4), wk.bk + ((size_t)(t0 + t) * H + h) * 4, 16);
+        }
+        if ((nt & 1u) && warp == (nt % NW)) {         // the idle partner of a last odd token
+            for (uint32_t c = lane; c < D; c += 32) { float* dt = d + nt * 3 * DP; dt[c] = 0.0f; dt[DP + c] = 0.0f; dt[2 * DP + c] = 1.0f; }
+            if (lane < NC) s_v[(stg * TC + nt) * NC + lane] = 0.0f;
+            if (lane < 4) s_bk[(stg * TC + nt) * 4 + lane] = 0.0f;
         }
         cp_commit();
     };
     fetch(0, 0);
-    const bool kind = l & 8, odd = l & 4;             // this lane ends up with S^T k (0) or S^T q (1) of column `odd`
+    const bool second = l & 8, isq = l & 4, odd = l & 2;      // the sum this lane ends up with: token, S^T q or S^T k, column
     for (uint32_t t0 = 0, stg = 0; t0 < rows; t0 += TC, stg ^= 1) {
         fetch(t0 + TC, stg ^ 1);
         cp_wait<1>();
         __syncthreads();
         const uint32_t nt = min(TC, rows - t0);
         const float* kqg = s_kqg + stg * TC * 3 * DP + l * 4;
-        uint64_t k[RPL / 2], q[RPL / 2], gd[RPL / 2];
-        auto load = [&](uint32_t t) {
-            const float* p = kqg + t * 3 * DP;
+        for (uint32_t t = 0; t < nt; t += 2) {
+            const float *p1 = kqg + t * 3 * DP, *p2 = p1 + 3 * DP;
+            const float4 bk1 = *(const float4*)(s_bk + (stg * TC + t) * 4), bk2 = *(const float4*)(s_bk + (stg * TC + t + 1) * 4);
+            const float2 v1 = *(const float2*)(s_v + (stg * TC + t) * NC + cl), v2 = *(const float2*)(s_v + (stg * TC + t + 1) * NC + cl);
+            uint64_t ka[RPL / 2], kb[RPL / 2], a1[2], b1[2], a2[2], b2[2];
 #pragma unroll
             for (int i = 0; i < RPL; i += 4) {
-                const ulonglong2 k2 = *(const ulonglong2*)(p + i * 16), q2 = *(const ulonglong2*)(p + DP + i * 16), g2 = *(const ulonglong2*)(p + 2 * DP + i * 16);
-                k[i / 2] = k2.x; k[i / 2 + 1] = k2.y;
-                q[i / 2] = q2.x; q[i / 2 + 1] = q2.y;
-                gd[i / 2] = g2.x; gd[i / 2 + 1] = g2.y;
-            }
-        };
-        load(0);
-        for (uint32_t t = 0; t < nt; t++) {
-            const float2 bk = *(const float2*)(s_bk + (stg * TC + t) * 2);
-            const float vm = s_v[(stg * TC + t) * NC + cl + odd];
-            uint64_t kc[RPL / 2], ak[2], aq[2];
-#pragma unroll
-            for (int i = 0; i < RPL / 2; i++) {
-                kc[i] = k[i];
+                const ulonglong2 k1 = *(const ulonglong2*)(p1 + i * 16), q1 = *(const ulonglong2*)(p1 + DP + i * 16), g1 = *(const ulonglong2*)(p1 + 2 * DP + i * 16);
+                const ulonglong2 k2 = *(const ulonglong2*)(p2 + i * 16), q2 = *(const ulonglong2*)(p2 + DP + i * 16), g2 = *(const ulonglong2*)(p2 + 2 * DP + i * 16);
+                ka[i / 2] = mul2(g2.x, k1.x); ka[i / 2 + 1] = mul2(g2.y, k1.y);
+                kb[i / 2] = k2.x; kb[i / 2 + 1] = k2.y;
 #pragma unroll
                 for (int c = 0; c < 2; c++) {
-                    S[i][c] = mul2(S[i][c], gd[i]);
-                    ak[c] = i == 0 ? mul2(S[0][c], k[0]) : fma2(S[i][c], k[i], ak[c]);
-                    aq[c] = i == 0 ? mul2(S[0][c], q[0]) : fma2(S[i][c], q[i], aq[c]);
+                    uint64_t x = mul2(S[i / 2][c], g1.x), y = mul2(S[i / 2 + 1][c], g1.y);
+                    a1[c] = i == 0 ? mul2(x, k1.x) : fma2(x, k1.x, a1[c]);
+                    b1[c] = i == 0 ? mul2(x, q1.x) : fma2(x, q1.x, b1[c]);
+                    a1[c] = fma2(y, k1.y, a1[c]);
+                    b1[c] = fma2(y, q1.y, b1[c]);
+                    x = mul2(x, g2.x); y = mul2(y, g2.y);
+                    a2[c] = i == 0 ? mul2(x, k2.x) : fma2(x, k2.x, a2[c]);
+                    b2[c] = i == 0 ? mul2(x, q2.x) : fma2(x, q2.x, b2[c]);
+                    a2[c] = fma2(y, k2.y, a2[c]);
+                    b2[c] = fma2(y, q2.y, b2[c]);
+                    S[i / 2][c] = x; S[i / 2 + 1][c] = y;
                 }
             }
-            if (t + 1 < nt) load(t + 1);
-            const float k0 = sum2(ak[0]), k1 = sum2(ak[1]), q0 = sum2(aq[0]), q1 = sum2(aq[1]);
-            const float e0 = (kind ? q0 : k0) + __shfl_xor_sync(0xffffffffu, kind ? k0 : q0, 8);
-            const float e1 = (kind ? q1 : k1) + __shfl_xor_sync(0xffffffffu, kind ? k1 : q1, 8);
-            float e = (odd ? e1 : e0) + __shfl_xor_sync(0xffffffffu, odd ? e0 : e1, 4);
-            e += __shfl_xor_sync(0xffffffffu, e, 2);
+            float e4[4], e2[2], e;
+            {
+                const float x0 = sum2(a1[0]), x1 = sum2(a1[1]), x2 = sum2(b1[0]), x3 = sum2(b1[1]);
+                const float y0 = sum2(a2[0]), y1 = sum2(a2[1]), y2 = sum2(b2[0]), y3 = sum2(b2[1]);
+                e4[0] = (second ? y0 : x0) + __shfl_xor_sync(0xffffffffu, second ? x0 : y0, 8);
+                e4[1] = (second ? y1 : x1) + __shfl_xor_sync(0xffffffffu, second ? x1 : y1, 8);
+                e4[2] = (second ? y2 : x2) + __shfl_xor_sync(0xffffffffu, second ? x2 : y2, 8);
+                e4[3] = (second ? y3 : x3) + __shfl_xor_sync(0xffffffffu, second ? x3 : y3, 8);
+            }
+            e2[0] = (isq ? e4[2] : e4[0]) + __shfl_xor_sync(0xffffffffu, isq ? e4[0] : e4[2], 4);
+            e2[1] = (isq ? e4[3] : e4[1]) + __shfl_xor_sync(0xffffffffu, isq ? e4[1] : e4[3], 4);
+            e = (odd ? e2[1] : e2[0]) + __shfl_xor_sync(0xffffffffu, odd ? e2[0] : e2[1], 2);
             e += __shfl_xor_sync(0xffffffffu, e, 1);
-            const float um = bk.x * (vm - e);         // u of column `odd`, in the lanes of kind 0
-            const float u0 = __shfl_sync(0xffffffffu, um, base), u1 = __shfl_sync(0xffffffffu, um, base | 4);
-            const uint64_t uu0 = pk2(u0, u0), uu1 = pk2(u1, u1);
+            // S^T k of both tokens and columns to every lane
+            const float s10 = __shfl_sync(0xffffffffu, e, base), s11 = __shfl_sync(0xffffffffu, e, base | 2);
+            const float s20 = __shfl_sync(0xffffffffu, e, base | 8), s21 = __shfl_sync(0xffffffffu, e, base | 10);
+            const float u10 = bk1.x * (v1.x - s10), u11 = bk1.x * (v1.y - s11);
+            const float u20 = bk2.x * (v2.x - fmaf(u10, bk2.z, s20)), u21 = bk2.x * (v2.y - fmaf(u11, bk2.z, s21));
+            const uint64_t w10 = pk2(u10, u10), w11 = pk2(u11, u11), w20 = pk2(u20, u20), w21 = pk2(u21, u21);
 #pragma unroll
             for (int i = 0; i < RPL / 2; i++) {
-                S[i][0] = fma2(kc[i], uu0, S[i][0]);
-                S[i][1] = fma2(kc[i], uu1, S[i][1]);
+                S[i][0] = fma2(kb[i], w20, fma2(ka[i], w10, S[i][0]));
+                S[i][1] = fma2(kb[i], w21, fma2(ka[i], w11, S[i][1]));
             }
-            if (kind && !(l & 3) && c0 + cl + odd < V) a.o[((size_t)(t0 + t) * H + h) * V + c0 + cl + odd] = fmaf(odd ? u1 : u0, bk.y, e);
+            if (isq && !(l & 1) && c0 + cl + odd < V && t + second < nt) {
+                const float u1 = odd ? u11 : u10, u2 = odd ? u21 : u20;
+                a.o[((size_t)(t0 + t + second) * H + h) * V + c0 + cl + odd] = second ? fmaf(u2, bk2.y, fmaf(u1, bk2.w, e)) : fmaf(u1, bk1.y, e);
+            }
         }
         __syncthreads();
     }
@@ -497,11 +534,20 @@ bool launch_step(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
     return rows == 1 ? launch_step_r<A, RPL, 1>(st, a, rows) : launch_step_r<A, RPL, (int)STEP_ROWS>(st, a, rows);
 }
 
+template <class A>
+void launch_prep(cudaStream_t st, const DeltaArgs& a, const DeltaWork& w, uint32_t rows) {
+    const dim3 grid((a.heads + 7) / 8, (rows + 1) / 2);
+    if (a.dim <= 64) launch_pdl(delta_prep_kernel<A, 2>, grid, dim3(256), 0, st, a, w, rows);
+    else if (a.dim <= 128) launch_pdl(delta_prep_kernel<A, 4>, grid, dim3(256), 0, st, a, w, rows);
+    else launch_pdl(delta_prep_kernel<A, 16>, grid, dim3(256), 0, st, a, w, rows);
+    g_launches++;
+}
+
 // Ordinary launch: CTAs that come up while the kernel before still holds SMs pile up on the ones it has left, and the
 // recurrence then runs at the pace of the fullest SM.
 template <int RPL, int NW, bool VEC>
 void launch_scan_t(cudaStream_t st, const DeltaArgs& a, const DeltaWork& w, uint32_t rows) {
-    const size_t smem = (size_t)2 * TC * (3 * 16 * RPL + NW * 4 + 2) * 4;
+    const size_t smem = (size_t)2 * TC * (3 * 16 * RPL + NW * 4 + 4) * 4;
     static int have[64] = {};
     ensure_dyn_smem(delta_scan_kernel<RPL, NW, VEC>, smem, have);
     delta_scan_kernel<RPL, NW, VEC><<<dim3((a.vdim + NW * 4 - 1) / (NW * 4), a.heads), NW * 32, smem, st>>>(a, w, rows);
@@ -527,15 +573,14 @@ void k_short_conv(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
 }
 
 size_t delta_work_floats(const DeltaArgs& a, uint32_t rows) {
-    return 2 * up4((size_t)rows * a.kv_heads * a.dim) + up4((size_t)rows * a.heads * a.dim) + up4((size_t)rows * a.heads * 2);
+    return 2 * up4((size_t)rows * a.kv_heads * a.dim) + up4((size_t)rows * a.heads * a.dim) + (size_t)rows * a.heads * 4;
 }
 
 void k_channel_delta(cudaStream_t st, const DeltaArgs& a, uint32_t rows) {
     if (!rows) return;
     const DeltaWork w = work_of(a, rows);
-    if (a.bf16) launch_pdl(delta_prep_kernel<ActBf16>, dim3(rows), dim3(256), (size_t)a.kv_heads * 4, st, a, w);
-    else launch_pdl(delta_prep_kernel<ActF32>, dim3(rows), dim3(256), (size_t)a.kv_heads * 4, st, a, w);
-    g_launches++;
+    if (a.bf16) launch_prep<ActBf16>(st, a, w, rows);
+    else launch_prep<ActF32>(st, a, w, rows);
     if (a.dim <= 64) launch_scan<4>(st, a, w, rows);
     else if (a.dim <= 128) launch_scan<8>(st, a, w, rows);
     else if (a.dim <= 256) launch_scan<16>(st, a, w, rows);
