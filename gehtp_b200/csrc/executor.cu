@@ -323,6 +323,8 @@ int status_message(unsigned int code, char* m, size_t mn) {
 // Ends a run: waits for the stream and turns a device-raised status into the
 // reference's error return.
 static int finish_run(char* err, size_t errn) {
+    // a launch the driver refused (not a fault of a kernel) shows here only
+    if (cudaError_t le = cudaGetLastError()) { cudaStreamSynchronize(g.stream); set_err(err, errn, cudaGetErrorString(le)); return -1; }
     cudaMemcpyAsync(g.h_status, g.d_status, sizeof(unsigned int), cudaMemcpyDeviceToHost, g.stream);
     cudaError_t ce = cudaStreamSynchronize(g.stream);
     if (ce != cudaSuccess) { set_err(err, errn, cudaGetErrorString(ce)); return -1; }

@@ -1,8 +1,9 @@
 """Ripidra: a decoder of latent-attention and channel-decay delta-rule layers, written as a row-count runlist.
 
-Each sublayer reads the residual stream itself and its output is RMS-normed before it is added; the norm weights are
-stored around zero. Layers may use the weights of an earlier layer with a cache or state of their own. The embedding
-table is also the head. Sizes and constants come from config.json and from tensor shapes.
+There is no norm in front of a sublayer: mixers and feed-forwards take the residual stream, and an RMS norm sits between
+their output and the addition (its weights are deviations from one). A layer may borrow another layer's weights while it
+keeps its own cache or state. Embedding and head are one table. Sizes and constants come from config.json and from
+tensor shapes.
 """
 from dataclasses import dataclass, field
 

@@ -93,7 +93,7 @@ enum {
  * OP_LINEAR         [x, w, y, rows, K, N, flags, x_col, x_stride]             y = act(x[:, x_col: x_col + K] . w^T), w bf16 [N, K];
  *                   flags: WT_LIN_*; x_stride 0 = K
  * OP_NORM_RESID     [y, w, x, x_out, act_out, rows, width, flags, eps_bits]   x_out = x + y / rms(y) * (b + w), w fp32;
- *                   flags: bit 0 b = 1 (weight stored around zero) else b = 0, bit 1 act_out is bf16, bit 2 y is bf16.
+ *                   flags: bit 0 b = 1 (weights are deviations from one) else b = 0, bit 1 act_out is bf16, bit 2 y is bf16.
  *                   x = 0: no residual; x_out / act_out = 0: not written
  * OP_PICK_ROWS      [x, idx, idx_off, out, rows, width]                       out[r] = x[idx[idx_off + r]] (fp32 rows, int32 idx)
  * OP_LATENT_APPEND  [y, norm_w, rope, q_out, gate_out, state, rows, heads, dim, rot, rank, eps_bits, flags]
