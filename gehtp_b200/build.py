@@ -38,6 +38,8 @@ UNITS = {
     "linear_rows.cu": [],
     "latent_attn.cu": [],
     "latent_prefill.cu": [],
+    "window_attn.cu": [],
+    "window_prefill.cu": [],
     "channel_delta.cu": [],
     "tp.cu": [],
     "tp_p2p.cu": [],

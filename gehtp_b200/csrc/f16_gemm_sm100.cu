@@ -26,7 +26,7 @@
 #include <cuda_runtime.h>
 #include "common.cuh"
 #include "launchers_rows.h"
-#include "rows_common.cuh"
+#include "linear_epi.cuh"
 #include "sm100_umma.cuh"
 #include "w4_stream.cuh"
 
@@ -54,69 +54,42 @@ struct __align__(8) FBarriers {
 
 __device__ __forceinline__ uint32_t pack2(float a, float b) { return (uint32_t)f2h(a) | ((uint32_t)f2h(b) << 16); }
 
-// Operand and output types of the kernel. EDGE: N need not be a multiple of the tile width nor K of 64 (the tensor
-// maps zero-fill what lies outside), the epilogue checks its columns; store8 writes 8 neighbouring outputs.
-struct IoF16 {                                    // the runlist's fp16 matmul
-    typedef uint16_t Out;
+// Epilogues of the kernel: the runlist's fp16 matmul here, the row-count projections' in linear_epi.cuh.
+struct EpiF16 {
+    uint16_t* y;                                  // rows 16-byte aligned: y is and ldy is a multiple of 8
+    uint32_t ldy;
+    __device__ __forceinline__ void quad(uint32_t m, uint32_t n, const float* v, uint32_t) const {
+        *(uint2*)(y + (size_t)m * ldy + n) = make_uint2(pack2(v[0], v[1]), pack2(v[2], v[3]));
+    }
+    __device__ __forceinline__ void chunk(uint32_t m, uint32_t n, const float (&f)[32], uint32_t) const {
+        uint16_t* d = y + (size_t)m * ldy + n;
+#pragma unroll
+        for (int q = 0; q < 4; q++) {
+            const float* v = f + 8 * q;
+            *(uint4*)(d + 8 * q) = make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7]));
+        }
+    }
+};
+// Operand type by epilogue. EDGE: N need not be a multiple of the tile width nor K of 64 (the tensor maps zero-fill what
+// lies outside), the epilogue checks its columns.
+template <class E> struct InOf {
+    static constexpr bool EDGE = true;
+    static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    static constexpr uint32_t IDESC = (1u << 7) | (1u << 10);      // A and B are bf16
+};
+template <> struct InOf<EpiF16> {
     static constexpr bool EDGE = false;
     static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
     static constexpr uint32_t IDESC = 0;
-    static __device__ __forceinline__ void store8(Out* p, const float* v, uint32_t) {
-        *(uint4*)p = make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7]));
-    }
-    static __device__ __forceinline__ void store4(Out* p, const float* v, uint32_t) { *(uint2*)p = make_uint2(pack2(v[0], v[1]), pack2(v[2], v[3])); }
-};
-template <bool RELU2>
-__device__ __forceinline__ float lin_act(float v) {
-    if (!RELU2) return v;
-    v = fmaxf(v, 0.0f);
-    return v * v;
-}
-constexpr uint32_t IDESC_BF16 = (1u << 7) | (1u << 10);      // A and B are bf16
-template <bool RELU2>
-struct IoBf16 {                                   // bf16 in, bf16 out
-    typedef uint16_t Out;
-    static constexpr bool EDGE = true;
-    static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-    static constexpr uint32_t IDESC = IDESC_BF16;
-    static __device__ __forceinline__ uint32_t pk(float a, float b) { return pack_bf2(lin_act<RELU2>(a), lin_act<RELU2>(b)); }
-    static __device__ __forceinline__ void store8(Out* p, const float* v, uint32_t left) {
-        if (left >= 8 && ((uintptr_t)p & 15u) == 0) { *(uint4*)p = make_uint4(pk(v[0], v[1]), pk(v[2], v[3]), pk(v[4], v[5]), pk(v[6], v[7])); return; }
-#pragma unroll
-        for (uint32_t i = 0; i < 8; i++) if (i < left) p[i] = f2bf(lin_act<RELU2>(v[i]));
-    }
-    static __device__ __forceinline__ void store4(Out* p, const float* v, uint32_t left) {
-#pragma unroll
-        for (uint32_t i = 0; i < 4; i++) if (i < left) p[i] = f2bf(lin_act<RELU2>(v[i]));
-    }
-};
-template <bool RELU2>
-struct IoBf16F32 {                                // bf16 in, fp32 out
-    typedef float Out;
-    static constexpr bool EDGE = true;
-    static constexpr CUtensorMapDataType MAP = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-    static constexpr uint32_t IDESC = IDESC_BF16;
-    static __device__ __forceinline__ void store4(Out* p, const float* v, uint32_t left) {
-        if (left >= 4 && ((uintptr_t)p & 15u) == 0) {
-            *(float4*)p = make_float4(lin_act<RELU2>(v[0]), lin_act<RELU2>(v[1]), lin_act<RELU2>(v[2]), lin_act<RELU2>(v[3]));
-            return;
-        }
-#pragma unroll
-        for (uint32_t i = 0; i < 4; i++) if (i < left) p[i] = lin_act<RELU2>(v[i]);
-    }
-    static __device__ __forceinline__ void store8(Out* p, const float* v, uint32_t left) {
-        store4(p, v, left);
-        if (left > 4) store4(p + 4, v + 4, left - 4);
-    }
 };
 
-// y rows are ldy elements apart (the SPLIT form writes N columns of a row of N_full).
-template <int MH, int BN, class IO>
+// fp16 outputs: rows ldy elements apart (the SPLIT form writes N columns of a row of N_full).
+template <int MH, int BN, class E>
 __global__ void __launch_bounds__(NTHREADS, 1)
 f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_w,
-                      typename IO::Out* __restrict__ y, uint32_t M, uint32_t K, uint32_t N, uint32_t ldy, unsigned int* status,
-                      uint32_t S, float* __restrict__ part) {
+                      const E epi, uint32_t M, uint32_t K, uint32_t N, unsigned int* status, uint32_t S, float* __restrict__ part) {
     using C = FCfg<MH, BN>;
+    using IO = InOf<E>;
     constexpr int STAGES = C::STAGES, NBUF = C::NBUF, A_BYTES = C::A_BYTES, B_BYTES = C::B_BYTES;
     constexpr uint32_t ACC_COLS = C::ACC_COLS, TMEM_COLS = C::TMEM_COLS;
     extern __shared__ unsigned char smem_raw[];
@@ -238,13 +211,10 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
                         for (int q = 0; q < 8; q++)
                             if (!IO::EDGE || n + 4 * q < np) dst[q] = make_uint4(v[4 * q], v[4 * q + 1], v[4 * q + 2], v[4 * q + 3]);
                     } else if (m < M) {
-                        typename IO::Out* dst = y + (size_t)m * ldy + n;     // fp16: 16-byte aligned, y is and ldy is a multiple of 8
                         float f[32];
 #pragma unroll
                         for (int q = 0; q < 32; q++) f[q] = __uint_as_float(v[q]);
-#pragma unroll
-                        for (int q = 0; q < 4; q++)
-                            if (!IO::EDGE || n + 8 * q < N) IO::store8(dst + 8 * q, f + 8 * q, IO::EDGE ? N - n - 8 * q : 8);
+                        if (!IO::EDGE || n < N) epi.chunk(m, n, f, N);
                     }
                 }
             }
@@ -272,10 +242,10 @@ bool make_map(CUtensorMap* tm, CUtensorMapDataType type, const uint16_t* base, u
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-// y[m][n] (rows ldy apart) = sum over the runs of part[run][m][n], in run order; 4 columns per thread
-template <class IO>
+// sum over the runs of part[run][m][n], in run order, to the epilogue; 4 columns per thread
+template <class E>
 __global__ void __launch_bounds__(256)
-f16_splitk_reduce_kernel(const float* __restrict__ part, typename IO::Out* __restrict__ y, uint32_t M, uint32_t N, uint32_t ldy, uint32_t S) {
+f16_splitk_reduce_kernel(const float* __restrict__ part, const E epi, uint32_t M, uint32_t N, uint32_t S) {
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const uint32_t nq = (N + 3) / 4;
@@ -289,7 +259,7 @@ f16_splitk_reduce_kernel(const float* __restrict__ part, typename IO::Out* __res
         const size_t m = i / nq;
         const uint32_t n = (uint32_t)(i % nq) * 4;
         const float v[4] = {acc.x, acc.y, acc.z, acc.w};
-        IO::store4(y + m * ldy + n, v, N - n);
+        epi.quad((uint32_t)m, n, v, N);
     }
 }
 
@@ -312,15 +282,16 @@ SplitScratch* split_scratch(cudaStream_t st, size_t need) {
     return &sc;
 }
 
-template <int MH, int BN, class IO>
-bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w, typename IO::Out* y, uint32_t M, uint32_t K, uint32_t N, uint32_t ldy,
+template <int MH, int BN, class E>
+bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w, const E& epi, uint32_t M, uint32_t K, uint32_t N,
             unsigned int* status, int sms) {
     using C = FCfg<MH, BN>;
+    using IO = InOf<E>;
     CUtensorMap ta, tw;
     if (!make_map(&ta, IO::MAP, a, M, K, lda, 128) || !make_map(&tw, IO::MAP, w, N, K, K, BN)) return false;
     const size_t smem = 1024 + (size_t)C::STAGES * (C::A_BYTES + C::B_BYTES) + sizeof(FBarriers) + 16;
     static int have[64] = {};
-    if (!ensure_dyn_smem(f16_gemm_sm100_kernel<MH, BN, IO>, smem, have)) return false;
+    if (!ensure_dyn_smem(f16_gemm_sm100_kernel<MH, BN, E>, smem, have)) return false;
     const uint32_t tiles = ((M + 128 * MH - 1) / (128 * MH)) * ((N + BN - 1) / BN), KG = (K + BK - 1) / BK;
     const uint32_t np = (N + 3) & ~3u;
     // Split K while the tiles alone leave SMs idle (same rule as the W4A16 GEMM): the divisor of K/64 that makes
@@ -342,7 +313,7 @@ bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w,
     }
     const uint32_t items = tiles * S;
     const uint32_t grid = items < (uint32_t)sms ? items : (uint32_t)sms;
-    if (launch_pdl(f16_gemm_sm100_kernel<MH, BN, IO>, dim3(grid), dim3(NTHREADS), smem, st, ta, tw, y, M, K, N, ldy, status, S, part) != cudaSuccess) {
+    if (launch_pdl(f16_gemm_sm100_kernel<MH, BN, E>, dim3(grid), dim3(NTHREADS), smem, st, ta, tw, epi, M, K, N, status, S, part) != cudaSuccess) {
         cudaGetLastError();
         return false;
     }
@@ -351,7 +322,7 @@ bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w,
         const size_t quads = (size_t)M * np / 4;
         uint32_t rg = (uint32_t)((quads + 255) / 256);
         if (rg > (uint32_t)sms * 8) rg = (uint32_t)sms * 8;
-        if (launch_pdl(f16_splitk_reduce_kernel<IO>, dim3(rg), dim3(256), 0, st, (const float*)part, y, M, N, ldy, S) != cudaSuccess) {
+        if (launch_pdl(f16_splitk_reduce_kernel<E>, dim3(rg), dim3(256), 0, st, (const float*)part, epi, M, N, S) != cudaSuccess) {
             cudaGetLastError();
             return false;
         }
@@ -490,9 +461,9 @@ bool launch_gemv(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint16_t
 }
 
 // tile shape by the number of tiles it gives
-template <class IO>
-bool launch_tiles(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w, typename IO::Out* y, uint32_t M, uint32_t K, uint32_t N,
-                  uint32_t ldy, unsigned int* status) {
+template <class E>
+bool launch_tiles(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w, const E& epi, uint32_t M, uint32_t K, uint32_t N,
+                  unsigned int* status) {
     static int sms_of[64] = {};
     int dev = 0;
     cudaGetDevice(&dev);
@@ -502,9 +473,9 @@ bool launch_tiles(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16
         if (sms <= 0) sms = 148;
     }
     const uint32_t t256 = ((M + 255) / 256) * ((N + 255) / 256), t128 = ((M + 255) / 256) * ((N + 127) / 128);
-    if ((IO::EDGE || N % 256 == 0) && M > 128 && t256 >= (uint32_t)sms) return launch<2, 256, IO>(st, a, lda, w, y, M, K, N, ldy, status, sms);
-    if (M > 128 && t128 >= (uint32_t)sms) return launch<2, 128, IO>(st, a, lda, w, y, M, K, N, ldy, status, sms);
-    return launch<1, 128, IO>(st, a, lda, w, y, M, K, N, ldy, status, sms);
+    if ((InOf<E>::EDGE || N % 256 == 0) && M > 128 && t256 >= (uint32_t)sms) return launch<2, 256, E>(st, a, lda, w, epi, M, K, N, status, sms);
+    if (M > 128 && t128 >= (uint32_t)sms) return launch<2, 128, E>(st, a, lda, w, epi, M, K, N, status, sms);
+    return launch<1, 128, E>(st, a, lda, w, epi, M, K, N, status, sms);
 }
 
 }  // namespace
@@ -520,7 +491,7 @@ bool k_matmul_f16_nk(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint
         return M <= 4 ? launch_gemv<4>(st, a, w, y, M, K, N, ldy) : launch_gemv<8>(st, a, w, y, M, K, N, ldy);
     }
     if (M < 128 || K % BK || N % 128 || (ldy & 7u) || ((uintptr_t)y & 15u)) return false;
-    return launch_tiles<IoF16>(st, a, K, w, y, M, K, N, ldy, status);
+    return launch_tiles(st, a, K, w, EpiF16{y, ldy}, M, K, N, status);
 }
 
 // The same kernel on bf16 operands with the outputs of a row-count projection: any N, K a multiple of 8 (16-byte rows),
@@ -528,11 +499,11 @@ bool k_matmul_f16_nk(cudaStream_t st, const uint16_t* a, const uint16_t* w, uint
 bool k_linear_sm100(cudaStream_t st, const LinearArgs& a, uint32_t M, unsigned int* status) {
     if (!a.x_bf16 || !M || (a.K & 7u) || (a.xs & 7u) || ((((uintptr_t)a.x) | ((uintptr_t)a.w)) & 15u)) return false;
     const uint16_t* x = (const uint16_t*)a.x;
-    if (a.y_bf16)
-        return a.relu2 ? launch_tiles<IoBf16<true>>(st, x, a.xs, a.w, (uint16_t*)a.y, M, a.K, a.N, a.ys, status)
-                       : launch_tiles<IoBf16<false>>(st, x, a.xs, a.w, (uint16_t*)a.y, M, a.K, a.N, a.ys, status);
-    return a.relu2 ? launch_tiles<IoBf16F32<true>>(st, x, a.xs, a.w, (float*)a.y, M, a.K, a.N, a.ys, status)
-                   : launch_tiles<IoBf16F32<false>>(st, x, a.xs, a.w, (float*)a.y, M, a.K, a.N, a.ys, status);
+    auto go = [&](auto epi) { return launch_tiles(st, x, a.xs, a.w, epi, M, a.K, a.N, status); };
+    if (a.tanh) return go(make_epi_tanh<ActBf16>(a.p, a.res, a.next, a.x_out, a.act, a.N, a.act_ld));
+    if (a.gelu_gate) return go(EpiGelu<true>{a.y, a.ys});
+    if (a.y_bf16) return a.relu2 ? go(EpiPlain<true, true>{a.y, a.ys, a.bias}) : go(EpiPlain<true, false>{a.y, a.ys, a.bias});
+    return a.relu2 ? go(EpiPlain<false, true>{a.y, a.ys, a.bias}) : go(EpiPlain<false, false>{a.y, a.ys, a.bias});
 }
 
 }  // namespace gehtp

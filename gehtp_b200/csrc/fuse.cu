@@ -19,6 +19,9 @@
 //                       untransposed tensor through a three-dimensional tensor map
 //   latent attention    LATENT_APPEND + LATENT_ATTEND of a row-count runlist -> for few rows: append and query absorption
 //                       in one kernel, split attention over the cached rows, merge with the value up-projection
+//   window attention    HEADS_APPEND + WINDOW_ATTEND of a row-count runlist -> for one row: one kernel
+//   tanh residual       LINEAR + TANH_RESID of a row-count runlist -> the projection's epilogue
+//   picked norm         PICK_ROWS + TANH_RESID of a row-count runlist -> one kernel
 //   delta rule          LINEAR x2 (low-rank decay, gate), SHORT_CONV, CHANNEL_DELTA, GATED_NORM -> for few rows: one kernel
 // and marks the data-movement ops whose result is a constant of the blob (fold_constants).
 //
@@ -56,6 +59,10 @@ int input_args(const wt_op& op, int out[8]) {
         add(0); add(1); break;
     case OP_BINARY_F16: add(0); add(1); if (op.args[4] == 8) add(2); break;
     case OP_SCATTER_ND_F16: add(0); add(1); add(2); break;
+    case OP_LINEAR: case OP_PICK_ROWS: case OP_SHORT_CONV: case OP_ARGMAX_ROWS: case OP_LATENT_APPEND: case OP_HEADS_APPEND: add(0); break;
+    case OP_NORM_RESID: case OP_TANH_RESID: case OP_GATED_NORM: add(0); add(2); break;
+    case OP_LATENT_ATTEND: case OP_WINDOW_ATTEND: add(0); add(1); break;
+    case OP_CHANNEL_DELTA: add(0); add(1); add(2); break;
     case OP_DELTA_CHUNK_F16: for (int i = 0; i < 5; i++) add(i); break;
     case OP_CONCAT_F16: for (uint32_t i = 0; i < op.args[10] && i < 4; i++) add((int)i); break;
     case OP_SILU_F16: case OP_UNARY_F16: case OP_SOFTMAX_F16: case OP_STRIDED_SLICE_F16: case OP_SPLIT_F16:
@@ -141,7 +148,9 @@ struct Span {
                              // 7 [head][row][d] -> [row][head * d] transposition in front of a W4A16 GEMM,
                              // 8 per-row SLICE + ARGMAX of a matrix joined by a CONCAT tree (greedy sampling of a batch),
                              // 9 latent append + attention of a row-count runlist,
-                             // 10 low-rank projections + convolution + delta rule + gated norm of a row-count runlist
+                             // 10 low-rank projections + convolution + delta rule + gated norm of a row-count runlist,
+                             // 11 projection + tanh norm into the residual stream, 12 append + window attention,
+                             // 13 picked rows + tanh norm, each of a row-count runlist
     uint32_t first, count;
     std::vector<uint32_t> ops;
     // attention
@@ -556,6 +565,46 @@ bool match_delta_step(const Graph& G, uint32_t i, Span& sp) {
     return true;
 }
 
+// LINEAR with fp32 output, read by the TANH_RESID behind it alone
+bool match_tanh_resid(const Graph& G, uint32_t i, Span& sp) {
+    const wt_blob* b = G.b;
+    if (i + 1 >= b->n_ops) return false;
+    const wt_op &li = b->ops[i], &tr = b->ops[i + 1];
+    if (li.opcode != OP_LINEAR || tr.opcode != OP_TANH_RESID) return false;
+    if (tr.args[0] != li.args[2] || tr.args[6] != li.args[3] || tr.args[7] != li.args[5] || li.args[9] || (tr.args[8] & 4u)) return false;
+    if (li.args[6] & ~WT_LIN_X_BF16) return false;
+    if (tr.args[5] && ((tr.args[8] >> 1) & 1u) != (li.args[6] & WT_LIN_X_BF16)) return false;      // act in the type of the input
+    if (tr.args[2] == li.args[0] || tr.args[3] == li.args[0] || tr.args[5] == li.args[0]) return false;   // other columns still read it
+    sp.kind = 11; sp.first = i; sp.count = 2; sp.ops = {i, i + 1};
+    return closed(G, sp.ops, {i + 1});
+}
+
+// HEADS_APPEND directly in front of the WINDOW_ATTEND of its state and queries
+bool match_window_step(const Graph& G, uint32_t i, Span& sp) {
+    const wt_blob* b = G.b;
+    if (i + 1 >= b->n_ops) return false;
+    const wt_op &ap = b->ops[i], &at = b->ops[i + 1];
+    if (ap.opcode != OP_HEADS_APPEND || at.opcode != OP_WINDOW_ATTEND) return false;
+    if (at.args[0] != ap.args[3] || at.args[2] != ap.args[4] || at.args[12] != ap.args[12] || at.args[13] != ap.args[14]) return false;
+    if (at.args[11] != 0xFFFFFFFFu && at.args[1] != ap.args[0]) return false;
+    for (int k = 4; k < 9; k++) if (at.args[k] != ap.args[k + 1]) return false;   // rows, heads, kv_heads, dim, vdim
+    sp.kind = 12; sp.first = i; sp.count = 2; sp.ops = {i, i + 1};
+    sp.keep = {i};                                        // runs of more rows take the two ops one after the other
+    return true;
+}
+
+// PICK_ROWS read by the norm behind it alone
+bool match_picked_norm(const Graph& G, uint32_t i, Span& sp) {
+    const wt_blob* b = G.b;
+    if (i + 1 >= b->n_ops) return false;
+    const wt_op &pk = b->ops[i], &tr = b->ops[i + 1];
+    if (pk.opcode != OP_PICK_ROWS || tr.opcode != OP_TANH_RESID) return false;
+    if (tr.args[0] != pk.args[3] || tr.args[6] != pk.args[4] || tr.args[7] != pk.args[5] || tr.args[2] || tr.args[3] || (tr.args[8] & 4u)) return false;
+    if (tr.args[5] == pk.args[0]) return false;
+    sp.kind = 13; sp.first = i; sp.count = 2; sp.ops = {i, i + 1};
+    return closed(G, sp.ops, {i + 1});
+}
+
 std::vector<Span> g_spans;
 float* g_attn_scratch = nullptr;
 std::map<std::pair<uint32_t, uint64_t>, uint8_t*> g_skip_maps;   // (mask slot, S<<32|Sk) -> device tile-skip bitmap
@@ -631,6 +680,10 @@ void fuse_analyze(const wt_blob* b, const std::vector<PlanOp>& meas, std::vector
     for (uint32_t i = 0; i + 4 < b->n_ops; i++) {
         Span sp{};
         if (!taken[i] && match_delta_step(G, i, sp)) claim(sp);
+    }
+    for (uint32_t i = 0; i + 1 < b->n_ops; i++) {
+        Span sp{};
+        if (!taken[i] && !taken[i + 1] && (match_tanh_resid(G, i, sp) || match_window_step(G, i, sp) || match_picked_norm(G, i, sp))) claim(sp);
     }
     // temps written only by interior ops of chains
     std::vector<int> writes_in(kMaxTemps, 0), writes_out(kMaxTemps, 0);
@@ -713,6 +766,32 @@ void fuse_materialize(const wt_blob* b) {
                 append(st);
                 attend(st);
             };
+        } else if (sp.kind == 11) {
+            const PlanOp& tr = g.plan[sp.first + 1];
+            if (!head.rows_args || !tr.rows_args) continue;
+            LinearArgs l = head.rows_args->lin;
+            const TanhResidArgs& t = tr.rows_args->tanh;
+            l.tanh = true; l.p = t.p; l.res = t.x; l.next = t.next; l.x_out = t.x_out; l.act = t.act; l.act_ld = t.act_ld;
+            head.fused = [=](cudaStream_t st) { k_linear(st, l, rows_of(l.rows_arg), false, g.d_status); };
+        } else if (sp.kind == 12) {
+            const PlanOp &ap = g.plan[sp.first], &at = g.plan[sp.first + 1];
+            if (!ap.launch || !at.launch) continue;
+            WindowArgs w = at.rows_args->win;
+            const WindowArgs& x = ap.rows_args->win;
+            w.y = x.y; w.norms = x.norms; w.rope = x.rope; w.rot = x.rot; w.eps = x.eps; w.positions = x.positions;
+            auto append = ap.launch, attend = at.launch;
+            head.fused = [=](cudaStream_t st) {
+                if (k_window_step(st, w, rows_of(w.rows_arg))) return;
+                append(st);
+                attend(st);
+            };
+        } else if (sp.kind == 13) {
+            const PlanOp& tr = g.plan[sp.first + 1];
+            if (!head.rows_args || !tr.rows_args) continue;
+            TanhResidArgs t = tr.rows_args->tanh;
+            const TanhResidArgs& p = head.rows_args->tanh;
+            t.y = p.y; t.idx = p.idx; t.y_rows = p.y_rows;
+            head.fused = [=](cudaStream_t st) { k_tanh_resid(st, t, rows_of(t.rows_arg)); };
         } else if (sp.kind == 10) {
             std::vector<std::function<void(cudaStream_t)>> parts;
             for (uint32_t k = 0; k < 5; k++) if (g.plan[sp.first + k].launch) parts.push_back(g.plan[sp.first + k].launch);

@@ -1,7 +1,7 @@
-// Row-wise pieces of the row-count runlists: embedding rows, RMS norm added to the residual stream, picked rows,
-// greedy choice, position counters. The residual stream and every norm are fp32.
+// Row-wise pieces of the row-count runlists: embedding rows, RMS norm or element-wise tanh norm added to the residual
+// stream, picked rows, greedy choice, position counters. The residual stream and every norm are fp32.
 #include "launchers_rows.h"
-#include "rows_common.cuh"
+#include "linear_epi.cuh"
 
 namespace gehtp {
 
@@ -9,7 +9,8 @@ namespace {
 
 template <class A>
 __global__ void __launch_bounds__(256)
-embed_rows_kernel(const uint16_t* __restrict__ table, const int32_t* ids, float* x, typename A::T* act, uint32_t width, uint32_t vocab) {
+embed_rows_kernel(const uint16_t* __restrict__ table, const int32_t* ids, float* x, typename A::T* act, uint32_t act_ld, uint32_t width,
+                  uint32_t vocab, float scale) {
     pdl_release();
     pdl_wait();
     const uint32_t r = blockIdx.x;
@@ -17,9 +18,9 @@ embed_rows_kernel(const uint16_t* __restrict__ table, const int32_t* ids, float*
     const bool ok = id >= 0 && (uint32_t)id < vocab;             // the host checks ids; a stray one reads nothing
     const uint16_t* src = table + (size_t)(ok ? id : 0) * width;
     for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = ok ? bf2f(__ldg(src + i)) : 0.0f;
+        const float v = ok ? bf2f(__ldg(src + i)) * scale : 0.0f;
         x[(size_t)r * width + i] = v;
-        if (act) A::st(act + (size_t)r * width + i, v);
+        if (act) A::st(act + (size_t)r * act_ld + i, v);
     }
 }
 
@@ -90,6 +91,31 @@ norm_resid_kernel(const typename Y::T* y, const float* __restrict__ w, const flo
     }
 }
 
+// Rows of y (or, with idx, the rows idx picks of it) through the epilogue of linear_epi.cuh, 4 columns per thread
+template <class Y, class A>
+__global__ void __launch_bounds__(256)
+tanh_resid_kernel(const typename Y::T* y, const int32_t* idx, uint32_t y_rows, const EpiTanh<A> epi, uint32_t width) {
+    pdl_release();
+    pdl_wait();
+    const uint32_t r = blockIdx.y, n = (blockIdx.x * 256 + threadIdx.x) * 4;
+    if (n >= width) return;
+    uint32_t src = r;
+    bool ok = true;
+    if (idx) { const int32_t s = idx[r]; ok = s >= 0 && (uint32_t)s < y_rows; src = ok ? (uint32_t)s : 0u; }
+    const typename Y::T* p = y + (size_t)src * width + n;
+    float v[4];
+    if (sizeof(typename Y::T) == 4 && width % 4 == 0) {
+        const float4 q = __ldcg((const float4*)p);
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    } else {
+#pragma unroll
+        for (uint32_t k = 0; k < 4; k++) v[k] = n + k < width ? Y::ld(p + k) : 0.0f;
+    }
+#pragma unroll
+    for (uint32_t k = 0; k < 4; k++) v[k] = ok ? v[k] : 0.0f;
+    epi.quad(r, n, v, width);
+}
+
 __global__ void __launch_bounds__(256)
 pick_rows_kernel(const float* x, const int32_t* idx, float* out, uint32_t width, uint32_t x_rows) {
     pdl_release();
@@ -133,6 +159,12 @@ __global__ void state_advance_kernel(uint32_t* counters, uint32_t n, uint32_t ro
 }
 
 template <class Y, class A>
+void launch_tanh(cudaStream_t st, const TanhResidArgs& a, uint32_t rows) {
+    launch_pdl(tanh_resid_kernel<Y, A>, dim3((a.width + 1023) / 1024, rows), dim3(256), 0, st, (const typename Y::T*)a.y, a.idx, a.y_rows,
+               make_epi_tanh<A>(a.p, a.x, a.next, a.x_out, a.act, a.width, a.act_ld), a.width);
+}
+
+template <class Y, class A>
 void launch_norm(cudaStream_t st, const NormResidArgs& a, uint32_t rows) {
     const uintptr_t al = (uintptr_t)a.y | (uintptr_t)a.x | (uintptr_t)a.x_out | (uintptr_t)a.act;
     const typename Y::T* y = (const typename Y::T*)a.y;
@@ -145,11 +177,12 @@ void launch_norm(cudaStream_t st, const NormResidArgs& a, uint32_t rows) {
 
 }  // namespace
 
-void k_embed_rows(cudaStream_t st, const uint16_t* table, const int32_t* ids, float* x, void* act, uint32_t rows, uint32_t width, uint32_t vocab, bool bf16) {
+void k_embed_rows(cudaStream_t st, const uint16_t* table, const int32_t* ids, float* x, void* act, uint32_t act_ld, uint32_t rows, uint32_t width,
+                  uint32_t vocab, float scale, bool bf16) {
     if (!rows) return;
     // ordinary launch: the first kernel of a run starts after everything of the run before
-    if (bf16) embed_rows_kernel<ActBf16><<<rows, 256, 0, st>>>(table, ids, x, (uint16_t*)act, width, vocab);
-    else embed_rows_kernel<ActF32><<<rows, 256, 0, st>>>(table, ids, x, (float*)act, width, vocab);
+    if (bf16) embed_rows_kernel<ActBf16><<<rows, 256, 0, st>>>(table, ids, x, (uint16_t*)act, act_ld, width, vocab, scale);
+    else embed_rows_kernel<ActF32><<<rows, 256, 0, st>>>(table, ids, x, (float*)act, act_ld, width, vocab, scale);
     g_launches++;
 }
 
@@ -157,6 +190,13 @@ void k_norm_resid(cudaStream_t st, const NormResidArgs& a, uint32_t rows) {
     if (!rows) return;
     if (a.y_bf16) { if (a.act_bf16) launch_norm<ActBf16, ActBf16>(st, a, rows); else launch_norm<ActBf16, ActF32>(st, a, rows); }
     else { if (a.act_bf16) launch_norm<ActF32, ActBf16>(st, a, rows); else launch_norm<ActF32, ActF32>(st, a, rows); }
+    g_launches++;
+}
+
+void k_tanh_resid(cudaStream_t st, const TanhResidArgs& a, uint32_t rows) {
+    if (!rows) return;
+    if (a.y_bf16) { if (a.act_bf16) launch_tanh<ActBf16, ActBf16>(st, a, rows); else launch_tanh<ActBf16, ActF32>(st, a, rows); }
+    else { if (a.act_bf16) launch_tanh<ActF32, ActBf16>(st, a, rows); else launch_tanh<ActF32, ActF32>(st, a, rows); }
     g_launches++;
 }
 

@@ -51,30 +51,40 @@ void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p) {
     case OP_EMBED_ROWS: {
         const uint32_t rows = a[4], width = a[5], vocab = a[6];
         const bool bf = a[7] == WT_DT_BF16;
-        if (bad_rows(rows) || !width || !vocab) FAIL("embed shape");
+        const float scale = from_bits(a[8]);
+        const uint32_t es = bf ? 2u : 4u, ld = a[9] ? a[9] : width, col = a[10];
+        if (bad_rows(rows) || !width || !vocab || (uint64_t)col + width > ld) FAIL("embed shape");
         if (slot_bytes(b, a[0]) != (uint64_t)vocab * width * 2u) FAIL("embed table size");
         const uint16_t* tab = (const uint16_t*)P.ref(a[0]);
         const int32_t* ids = (const int32_t*)P.ref(a[1]);
         if ((a[1] & 0x8000u) && slot_bytes(b, a[1]) < (uint64_t)max_of(rows) * 4u) FAIL("embed ids too short");
         float* x = (float*)temp_rows(P, a[2], rows, (uint64_t)width * 4u, p);
-        void* act = a[3] ? (void*)temp_rows(P, a[3], rows, (uint64_t)width * (bf ? 2u : 4u), p) : nullptr;
+        uint8_t* act = a[3] ? temp_rows(P, a[3], rows, (uint64_t)ld * es, p) : nullptr;
         if (!tab || !ids || !x || (a[3] && !act)) FAIL("embed ref fail");
-        if (P.build) p.launch = [=](cudaStream_t st) { k_embed_rows(st, tab, ids, x, act, rows_of(rows), width, vocab, bf); };
+        if (act) act += (size_t)col * es;
+        if (P.build) p.launch = [=](cudaStream_t st) { k_embed_rows(st, tab, ids, x, act, ld, rows_of(rows), width, vocab, scale, bf); };
         return;
     }
     case OP_LINEAR: {
         const uint32_t rows = a[3], K = a[4], N = a[5], fl = a[6], xc = a[7];
         LinearArgs l{};
         l.K = K; l.N = N; l.xs = a[8] ? a[8] : K; l.ys = N; l.rows_arg = rows;
-        l.x_bf16 = fl & WT_LIN_X_BF16; l.y_bf16 = fl & WT_LIN_Y_BF16; l.relu2 = fl & WT_LIN_RELU2;
+        l.x_bf16 = fl & WT_LIN_X_BF16; l.y_bf16 = fl & WT_LIN_Y_BF16; l.relu2 = fl & WT_LIN_RELU2; l.gelu_gate = fl & WT_LIN_GELU_GATE;
+        if (l.y_bf16 && !l.x_bf16) FAIL("linear: bf16 output of fp32 input");
+        if (l.gelu_gate) {
+            if ((N & 1u) || l.relu2 || a[9] || l.y_bf16 != l.x_bf16) FAIL("linear: gated form n%u flags %u", N, fl);
+            l.ys = N / 2;
+        }
         const uint32_t xe = l.x_bf16 ? 2u : 4u;
         if (bad_rows(rows) || !K || !N || (uint64_t)xc + K > l.xs) FAIL("linear shape k%u n%u col%u stride%u", K, N, xc, l.xs);
         if (slot_bytes(b, a[1]) != (uint64_t)K * N * 2u) FAIL("linear weight size");
         const uint8_t* x = P.ref(a[0]);
         if (!temp_holds(P, a[0], (uint64_t)max_of(rows) * l.xs * xe)) FAIL("linear input too small");
         l.w = (const uint16_t*)P.ref(a[1]);
-        l.y = temp_rows(P, a[2], rows, (uint64_t)N * (l.y_bf16 ? 2u : 4u), p);
-        if (!x || !l.w || !l.y) FAIL("linear ref fail");
+        l.bias = a[9] ? (const float*)P.ref(a[9]) : nullptr;
+        if (a[9] && slot_bytes(b, a[9]) != (uint64_t)N * 4u) FAIL("linear bias size");
+        l.y = temp_rows(P, a[2], rows, (uint64_t)l.ys * (l.y_bf16 ? 2u : 4u), p);
+        if (!x || !l.w || !l.y || (a[9] && !l.bias)) FAIL("linear ref fail");
         l.x = x + (size_t)xc * xe;
         p.engine = WT_ENG_HMX;
         p.rows_args->lin = l;
@@ -99,6 +109,29 @@ void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p) {
         if (P.build) p.launch = [=](cudaStream_t st) { k_norm_resid(st, n, rows_of(rows)); };
         return;
     }
+    case OP_TANH_RESID: {
+        TanhResidArgs n{};
+        const uint32_t rows = a[6], fl = a[8], col = a[10];
+        n.width = a[7]; n.rows_arg = rows; n.act_bf16 = fl & 2u; n.y_bf16 = fl & 4u; n.act_ld = a[9] ? a[9] : n.width;
+        const uint32_t es = n.act_bf16 ? 2u : 4u;
+        const uint64_t pb = (4u + 2u * (uint64_t)n.width) * 4u;
+        if (bad_rows(rows) || !n.width || (uint64_t)col + n.width > n.act_ld) FAIL("tanh norm shape");
+        if ((a[1] && slot_bytes(b, a[1]) != pb) || (a[4] && slot_bytes(b, a[4]) != pb)) FAIL("tanh norm parameter size");
+        n.y = P.ref(a[0]);
+        if (!n.y || !temp_holds(P, a[0], (uint64_t)max_of(rows) * n.width * (n.y_bf16 ? 2u : 4u))) FAIL("tanh norm input too small");
+        if (a[1]) { n.p = (const float*)P.ref(a[1]); if (!n.p) FAIL("tanh norm ref fail"); }
+        if (a[4]) { n.next = (const float*)P.ref(a[4]); if (!n.next) FAIL("tanh norm ref fail"); }
+        if (a[2]) { n.x = (const float*)P.ref(a[2]); if (!n.x || !temp_holds(P, a[2], (uint64_t)max_of(rows) * n.width * 4u)) FAIL("tanh norm residual ref fail"); }
+        if (a[3]) { n.x_out = (float*)temp_rows(P, a[3], rows, (uint64_t)n.width * 4u, p); if (!n.x_out) FAIL("tanh norm out fail"); }
+        if (a[5]) {
+            uint8_t* act = temp_rows(P, a[5], rows, (uint64_t)n.act_ld * es, p);
+            if (!act) FAIL("tanh norm out fail");
+            n.act = act + (size_t)col * es;
+        }
+        p.rows_args->tanh = n;
+        if (P.build) p.launch = [=](cudaStream_t st) { k_tanh_resid(st, n, rows_of(rows)); };
+        return;
+    }
     case OP_PICK_ROWS: {
         const uint32_t rows = a[4], width = a[5];
         if (bad_rows(rows) || !width) FAIL("pick shape");
@@ -109,6 +142,8 @@ void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p) {
         float* out = (float*)temp_rows(P, a[3], rows, (uint64_t)width * 4u, p);
         if (!x || !idx || !out || !x_rows) FAIL("pick ref fail");
         const int32_t* id0 = idx + a[2];
+        TanhResidArgs& t = p.rows_args->tanh;             // the picked rows, for a norm fused behind
+        t.y = x; t.idx = id0; t.y_rows = x_rows;
         if (P.build) p.launch = [=](cudaStream_t st) { k_pick_rows(st, x, id0, out, rows_of(rows), width, x_rows); };
         return;
     }
@@ -159,6 +194,55 @@ void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p) {
             };
         }
         p.rows_args->lat = l;
+        return;
+    }
+    case OP_HEADS_APPEND: case OP_WINDOW_ATTEND: {
+        const bool app = op.opcode == OP_HEADS_APPEND;
+        WindowArgs w{};
+        const uint32_t rows = w.rows_arg = a[app ? 5 : 4];
+        w.heads = a[app ? 6 : 5]; w.kv_heads = a[app ? 7 : 6]; w.dim = a[app ? 8 : 7]; w.vdim = a[app ? 9 : 8];
+        w.y_cols = a[12]; w.bf16 = a[app ? 14 : 13] == WT_DT_BF16;
+        const uint32_t es = w.bf16 ? 2u : 4u;
+        const uint64_t mr = max_of(rows), qrow = (uint64_t)w.heads * w.dim, orow = (uint64_t)w.heads * w.vdim;
+        if (bad_rows(rows) || !w.heads || !w.kv_heads || w.heads % w.kv_heads || !w.dim || !w.vdim) FAIL("window heads shape");
+        const int si = state_index(app ? a[4] : a[2]);
+        if (si < 0) FAIL("window state ref bad");
+        const uint32_t row_bytes = w.row() * es;
+        if (g.st_bytes[si] % row_bytes || g.st_bytes[si] / row_bytes < mr) FAIL("window state %d has %u bytes, rows of %u", si, g.st_bytes[si], row_bytes);
+        KvGeom& kv = g.kv[si];
+        if (kv.ready && kv.posmap) FAIL("window state %d is a KV ring of another kind", si);
+        w.state = g.st_buf[si]; w.counter = g.d_st_count + si; w.ring = g.st_bytes[si] / row_bytes; w.state_idx = (uint32_t)si; w.status = g.d_status;
+        if (app) {
+            w.rot = a[10]; w.eps = from_bits(a[11]); w.positions = a[13];
+            if ((w.rot & 1u) || w.rot > w.dim || !w.positions) FAIL("window rotation %u of %u", w.rot, w.dim);
+            if (w.y_cols < w.min_cols() || !temp_holds(P, a[0], mr * w.y_cols * es)) FAIL("window input too small");
+            if (a[1] && slot_bytes(b, a[1]) != (uint64_t)w.dim * 8u) FAIL("window norm weight size");
+            if (w.rot && slot_bytes(b, a[2]) < (uint64_t)w.positions * w.rot * 4u) FAIL("window rotary table too short");
+            w.y = P.ref(a[0]);
+            w.norms = a[1] ? (const float*)P.ref(a[1]) : nullptr;
+            w.rope = w.rot ? (const float*)P.ref(a[2]) : nullptr;
+            w.q = temp_rows(P, a[3], rows, qrow * es, p);
+            if (!w.y || (a[1] && !w.norms) || (w.rot && !w.rope) || !w.q) FAIL("window ref fail");
+            kv.ready = true; kv.slot_bytes = row_bytes; kv.nslots = w.positions;      // room is a matter of positions, not of ring rows
+            p.pos_append_state = si;
+            if (P.build) p.launch = [=](cudaStream_t st) { k_heads_append(st, w, rows_of(rows)); };
+        } else {
+            w.window = a[9]; w.scale = from_bits(a[10]); w.gate_col = a[11];
+            const bool gate = w.gate_col != 0xFFFFFFFFu;
+            if (!w.window) FAIL("window of no positions");
+            // a run's rows are appended before they attend: the ring holds them and the windows behind the first of them,
+            // unless no position is ever overwritten
+            if (kv.ready && kv.nslots > w.ring && (uint64_t)w.window - 1u + mr > w.ring) FAIL("window %u and %llu rows exceed a ring of %u", w.window, (unsigned long long)mr, w.ring);
+            if (gate && (uint64_t)w.gate_col + orow > w.y_cols) FAIL("window gate columns");
+            w.q = (void*)P.ref(a[0]);
+            if (!w.q || !temp_holds(P, a[0], mr * qrow * es)) FAIL("window input too small");
+            if (gate) { w.y = P.ref(a[1]); if (!w.y || !temp_holds(P, a[1], mr * w.y_cols * es)) FAIL("window gate too small"); }
+            w.out = temp_rows(P, a[3], rows, orow * es, p);
+            if (!w.out) FAIL("window ref fail");
+            p.engine = WT_ENG_HMX;
+            if (P.build) p.launch = [=](cudaStream_t st) { k_window_attend(st, w, rows_of(rows), !g.opt_fuse || g.exact_ops); };
+        }
+        p.rows_args->win = w;
         return;
     }
     case OP_SHORT_CONV: {

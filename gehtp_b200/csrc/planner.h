@@ -105,7 +105,7 @@ struct Planner {
         p.rc = -1; p.err = _m; return;                       \
     } while (0)
 
-// plan_rows.cu: opcodes OP_EMBED_ROWS .. OP_STATE_ADVANCE
+// plan_rows.cu: opcodes OP_EMBED_ROWS .. OP_WINDOW_ATTEND
 void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p);
 
 }  // namespace gehtp

@@ -64,8 +64,9 @@ const OpInfo* op_info(uint16_t opcode) {
     }
     // the executor's own row-count ops
     static const OpInfo rows_tab[OP_ROWS_END - OP_EMBED_ROWS] = {
-        {8, bits({0, 1})}, {9, bits({0, 1})}, {9, bits({0, 1, 2})}, {6, bits({0, 1})}, {13, bits({0, 1, 2})},
+        {11, bits({0, 1})}, {10, bits({0, 1, 9})}, {9, bits({0, 1, 2})}, {6, bits({0, 1})}, {13, bits({0, 1, 2})},
         {14, bits({3})}, {9, bits({0, 1})}, {16, bits({3, 4})}, {9, bits({1})}, {4, 0}, {3, 0},
+        {11, bits({1, 4})}, {15, bits({1, 2})}, {14, 0},
     };
     if (opcode >= OP_EMBED_ROWS && opcode < OP_ROWS_END) return &rows_tab[opcode - OP_EMBED_ROWS];
     if (opcode >= sizeof(tab) / sizeof(tab[0]) || tab[opcode].arity < 0) return nullptr;

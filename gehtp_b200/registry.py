@@ -2,13 +2,14 @@
 shapes of the synthetic benchmark models."""
 import os
 
-from . import ripidra
+from . import ripidra, supevik
 from .checkpoint import Tensors, read_config
 from .runlists import QWEN3_0P6B, QWEN3_4B
 
 # architecture -> (configuration from config.json, builder(config, tensors, dtype, max_tokens, max_rows, max_sel))
 ARCHITECTURES = {
     "Ripidra": (ripidra.RipidraConfig.from_json, ripidra.build_runlist),
+    "Supevik": (supevik.SupevikConfig.from_json, supevik.build_runlist),
 }
 # synthetic decoder shapes (seeded weights, runlists.py)
 SHAPES = {c.name: c for c in (QWEN3_0P6B, QWEN3_4B)}

@@ -1,18 +1,20 @@
 """Row-count runlists: one op list that runs any number of token rows of a sequence from the states earlier runs left
 (prompts whole or in portions, and single decoded tokens), written with the executor's own row ops.
 
-`RowsEmitter` holds the mechanisms - projections, norms on the residual stream, latent attention, the delta rule with a
-decay per key channel, dense feed-forwards, the picked-row head - each with its sizes and constants as arguments; a
-model design (ripidra.py) strings them together. Activations are bf16 or fp32, weights bf16, the residual stream fp32.
+`RowsEmitter` holds the mechanisms - projections, norms on the residual stream, latent attention, grouped-query attention
+over a window, the delta rule with a decay per key channel, dense feed-forwards, the picked-row head - each with its sizes
+and constants as arguments; a model design (ripidra.py, supevik.py) strings them together. Activations are bf16 or fp32,
+weights bf16, the residual stream fp32.
 
 Temps are named and reused from layer to layer: a layer's intermediate faces share the memory of the layer before.
 """
+import math
 import struct
 
 import numpy as np
 
 from .checkpoint import bf16_to_f32
-from .wtop import COL_ALIGN, DT_BF16, DT_F32, LIN_RELU2, LIN_X_BF16, LIN_Y_BF16, OP, ROWS_AUTO, S, SEL_AUTO, ST, BlobBuilder
+from .wtop import COL_ALIGN, DT_BF16, DT_F32, LIN_GELU_GATE, LIN_RELU2, LIN_X_BF16, LIN_Y_BF16, OP, ROWS_AUTO, S, SEL_AUTO, ST, BlobBuilder
 
 
 def bits(x):
@@ -47,6 +49,30 @@ def rope_pairs(positions, dims, base):
     """fp32 [positions][dims / 2][cos, sin] for neighbouring components turned by p * base^(-2i / dims)."""
     ang = np.arange(positions, dtype=np.float64)[:, None] * np.float64(base) ** (-np.arange(0, dims, 2, dtype=np.float64) / dims)
     return np.stack([np.cos(ang), np.sin(ang)], axis=-1).astype(np.float32)
+
+
+def yarn_scaling(dims, base, factor, original, fast, slow):
+    """(factor on each pair's angle, factor on cosine and sine) of YaRN context extension: pairs that turn more than `fast`
+    times over the original context keep their angle, those below `slow` turns have it divided by `factor`."""
+    def at(turns):
+        return dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), dims - 1)
+    ramp = np.clip((np.arange(dims // 2) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return ramp / factor + (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
+def rope_halves(positions, dims, base, scaling=None):
+    """fp32 [positions][dims / 2][cos, sin] for components i and i + dims / 2 turned by p * base^(-2i / dims); scaling:
+    the arguments of yarn_scaling by name."""
+    f, mag = np.float64(base) ** (-np.arange(0, dims, 2, dtype=np.float64) / dims), 1.0
+    if scaling:
+        by, mag = yarn_scaling(dims, base, scaling["factor"], scaling["original"], scaling["fast"], scaling["slow"])
+        f = f * by
+    ang = np.arange(positions, dtype=np.float64)[:, None] * f
+    return (np.stack([np.cos(ang), np.sin(ang)], axis=-1) * mag).astype(np.float32)
+
+
+RING_ALIGN = 128        # rows of a position ring are a multiple of the largest tile that is read from it
 
 
 class RowsEmitter:
@@ -97,18 +123,35 @@ class RowsEmitter:
         return self.b.add_op(opcode, args)
 
     # ---- single ops
-    def embed(self, table, vocab, width):
-        self.op(OP.EMBED_ROWS, [table, S(self.face), self.temp("x"), self.temp("act") if self.bf16 else 0, ROWS_AUTO, width, vocab, self.dt])
+    def embed(self, table, vocab, width, scale=1.0, act="act", col=0, stride=0):
+        """x = table rows * scale; their activation copy goes to columns `col` .. of temp `act` (None: no copy)."""
+        copy = self.temp(act) if act and (self.bf16 or act != "act") else 0
+        self.op(OP.EMBED_ROWS, [table, S(self.face), self.temp("x"), copy, ROWS_AUTO, width, vocab, self.dt, bits(scale), stride, col])
 
     def act(self):
         """The residual stream as projections read it: its bf16 copy, or the stream itself in fp32."""
         return self.temp("act") if self.bf16 else self.temp("x")
 
-    def linear(self, x, w, out, K, N, y_act=True, relu2=False, rows=ROWS_AUTO, col=0, stride=0):
+    def linear(self, x, w, out, K, N, y_act=True, relu2=False, rows=ROWS_AUTO, col=0, stride=0, bias=0, gelu_gate=False):
         fl = (LIN_X_BF16 if self.bf16 else 0) | (LIN_Y_BF16 if self.bf16 and y_act else 0) | (LIN_RELU2 if relu2 else 0)
         t = self.temp(out)
-        self.op(OP.LINEAR, [x, w, t, rows, K, N, fl, col, stride])
+        self.op(OP.LINEAR, [x, w, t, rows, K, N, fl | (LIN_GELU_GATE if gelu_gate else 0), col, stride, bias])
         return t
+
+    def tanh_params(self, key, alpha, w, b):
+        """Slot of an element-wise norm tanh(alpha z) w + b; arguments: zero-argument callables giving bf16 bits."""
+        def make():
+            a, w_, b_ = (bf16_to_f32(np.asarray(f())).reshape(-1) for f in (alpha, w, b))
+            if a.size != 1:
+                raise ValueError("%s: %d factors in front of tanh, expected one" % (key, a.size))
+            return np.concatenate([a, np.zeros(3, np.float32), w_, b_])
+        return self.slot((key, "tanh"), make)
+
+    def tanh_resid(self, y, width, p=0, add=True, to_x=True, then=0, act="act", col=0, stride=0, rows=ROWS_AUTO):
+        """x <- x + t(y, p) (add=False: t(y, p)); temp `act` (None: not written) gets t(x, then) from column `col` on."""
+        x = self.temp("x")
+        self.op(OP.TANH_RESID, [y, p, x if add else 0, x if to_x else 0, then, self.temp(act) if act else 0, rows, width,
+                                2 if self.bf16 else 0, stride, col])
 
     def add_norm(self, y, w, width, eps, about_one):
         """x <- x + norm(y), and the activation copy of x."""
@@ -130,6 +173,35 @@ class RowsEmitter:
         self.op(OP.LATENT_APPEND, [y, nw, self.rope_table(rot, base), q, gate, st, ROWS_AUTO, heads, dim, rot, rank, bits(eps), self.dt])
         self.op(OP.LATENT_ATTEND, [q, gate, st, w_kv, out, self.temp("work"), ROWS_AUTO, heads, dim, rot, vdim, rank, bits(scale), self.dt])
         return self.linear(out, w_o, "mix", heads * vdim, width, y_act=False)
+
+    def window_attention(self, key, x, width, heads, kv_heads, dim, vdim, window, rot, scale, eps, w):
+        """Grouped-query attention of rows x over the last `window` positions. rot: {dims, base, scaling}. w: q, k, v, g, o
+        and the biases q_b, k_b, v_b, the head norms q_norm, k_norm (None where the design has none; zero-argument callables)."""
+        at, cols = [], 0
+        for n in (heads * dim, kv_heads * dim, kv_heads * vdim) + ((heads * vdim,) if w["g"] else ()):
+            at.append(cols)
+            cols += up(n)
+
+        def bias():
+            out = np.zeros(cols, np.float32)
+            for a, n in zip(at, ("q_b", "k_b", "v_b")):
+                v = bf16_to_f32(w[n]())
+                out[a:a + v.size] = v
+            return out
+        w_in = self.slot((key, "in"), lambda: join_rows([w[n]() for n in "qkvg" if w[n]])[0])
+        b_in = self.slot((key, "bias"), bias) if w["q_b"] else 0
+        norms = self.slot((key, "norms"), lambda: bf16_to_f32(np.concatenate([w["q_norm"](), w["k_norm"]()]))) if w["q_norm"] else 0
+        dims = rot["dims"] if rot else 0
+        table = self.slot(("halves", dims, float(rot["base"]), tuple(sorted((rot.get("scaling") or {}).items()))),
+                          lambda: rope_halves(self.nslots, dims, rot["base"], rot.get("scaling"))) if dims else 0
+        row = up(kv_heads * (dim + vdim))
+        ring = min(up(self.nslots, RING_ALIGN), up(window - 1 + self.max_rows, RING_ALIGN))
+        st = self._state("cache", ring * row * self.es)
+        y = self.linear(x, w_in, "proj", width, cols, bias=b_in)
+        q, out = self.temp("q"), self.temp("heads")
+        self.op(OP.HEADS_APPEND, [y, norms, table, q, st, ROWS_AUTO, heads, kv_heads, dim, vdim, dims, bits(eps), cols, self.nslots, self.dt])
+        self.op(OP.WINDOW_ATTEND, [q, y, st, out, ROWS_AUTO, heads, kv_heads, dim, vdim, window, bits(scale), at[3] if w["g"] else 0xFFFFFFFF, cols, self.dt])
+        return self.linear(out, self.slot((key, "o"), w["o"]), "mix", heads * vdim, width, y_act=False)
 
     def channel_delta(self, key, width, heads, kv_heads, dim, vdim, taps, rank_a, rank_g, eps, w):
         """w: q, k, v, q_conv, k_conv, v_conv, b, a_log, norm, a1, a2, dt_bias, g1, g2, o."""
@@ -162,15 +234,34 @@ class RowsEmitter:
         h = self.linear(self.act(), self.slot((key, "up"), w["up"]), "ff", width, ff, relu2=True)
         return self.linear(h, self.slot((key, "down"), w["down"]), "mix", ff, width, y_act=False)
 
-    def head(self, norm_w, table, vocab, width, eps, about_one):
-        """Picked rows -> norm -> logits (fp32) and the greedy choice."""
-        p, h = self.temp("picked"), self.temp("picked_act")
+    def dense_gelu_gate(self, key, x, width, ff, w):
+        """(gelu(gate x) * up x) through `down`; w: gate, up, down."""
+        w_in = self.slot((key, "gate_up"), lambda: np.stack([w["gate"](), w["up"]()], axis=1).reshape(2 * ff, width))
+        h = self.linear(x, w_in, "ff", width, 2 * ff, gelu_gate=True)
+        return self.linear(h, self.slot((key, "down"), w["down"]), "mix", ff, width, y_act=False)
+
+    def pick(self, width):
+        p = self.temp("picked")
         self.op(OP.PICK_ROWS, [self.temp("x"), S(self.face), self.max_rows, p, SEL_AUTO, width])
-        self.op(OP.NORM_RESID, [p, norm_w, 0, 0, h, SEL_AUTO, width, (1 if about_one else 0) | (2 if self.bf16 else 0), bits(eps)])
+        return p
+
+    def choose(self, h, table, vocab, width):
+        """Logits (fp32) of picked rows h and the greedy choice."""
         logits = self.linear(h, table, "logits", width, vocab, y_act=False, rows=SEL_AUTO)
         tok = self.temp("token")
         self.op(OP.ARGMAX_ROWS, [logits, tok, SEL_AUTO, vocab])
         return logits, tok
+
+    def tanh_head(self, p, table, vocab, width):
+        """Picked rows -> element-wise norm -> logits and the greedy choice."""
+        self.tanh_resid(self.pick(width), width, add=False, to_x=False, then=p, act="picked_act", rows=SEL_AUTO)
+        return self.choose(self.temp("picked_act"), table, vocab, width)
+
+    def head(self, norm_w, table, vocab, width, eps, about_one):
+        """Picked rows -> norm -> logits (fp32) and the greedy choice."""
+        p, h = self.pick(width), self.temp("picked_act")
+        self.op(OP.NORM_RESID, [p, norm_w, 0, 0, h, SEL_AUTO, width, (1 if about_one else 0) | (2 if self.bf16 else 0), bits(eps)])
+        return self.choose(h, table, vocab, width)
 
     def finish(self):
         """Advances the counters, numbers the states, serialises."""

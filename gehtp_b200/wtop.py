@@ -17,7 +17,7 @@ SLOT_EXT_WGT, SLOT_STATE, KV_POS_AUTO = 0xFFFFFFFC, 0xFFFFFFFB, 0xFFFFFFFA
 # row-count runlists (this executor's own): limits slot, and the row arguments that follow the run
 SLOT_ROWS, ROWS_AUTO, SEL_AUTO = 0xFFFFFFF7, 0xFFFFFFF9, 0xFFFFFFF8
 DT_F32, DT_BF16 = 0, 1
-LIN_X_BF16, LIN_Y_BF16, LIN_RELU2 = 1, 2, 16
+LIN_X_BF16, LIN_Y_BF16, LIN_RELU2, LIN_GELU_GATE = 1, 2, 16, 32
 COL_ALIGN = 8
 
 
@@ -29,12 +29,14 @@ class OP:
     DMA, PAD, MATMUL_F16_SPLIT = 33, 34, 35
     EMBED_ROWS, LINEAR, NORM_RESID, PICK_ROWS, LATENT_APPEND, LATENT_ATTEND = range(0x140, 0x146)
     SHORT_CONV, CHANNEL_DELTA, GATED_NORM, ARGMAX_ROWS, STATE_ADVANCE = range(0x146, 0x14B)
+    TANH_RESID, HEADS_APPEND, WINDOW_ATTEND = range(0x14B, 0x14E)
 
 
 ARITY = {0: 0, 1: 6, 2: 4, 3: 1, 4: 3, 5: 15, 6: 13, 7: 4, 8: 4, 9: 4, 10: 6, 11: 4, 12: 5, 13: 4,
          14: 16, 15: 16, 16: 16, 17: 9, 18: 7, 19: 6, 20: 15, 21: 3, 22: 4, 23: 7, 24: 7, 25: 5,
          26: 12, 27: 8, 28: 14, 29: 6, 30: 12, 33: 8, 34: 7, 35: 9,
-         0x140: 8, 0x141: 9, 0x142: 9, 0x143: 6, 0x144: 13, 0x145: 14, 0x146: 9, 0x147: 16, 0x148: 9, 0x149: 4, 0x14A: 3}
+         0x140: 11, 0x141: 10, 0x142: 9, 0x143: 6, 0x144: 13, 0x145: 14, 0x146: 9, 0x147: 16, 0x148: 9, 0x149: 4, 0x14A: 3,
+         0x14B: 11, 0x14C: 15, 0x14D: 14}
 
 
 # argument positions that name the temp(s) an op writes
@@ -42,7 +44,7 @@ _OUT_ARGS = {1: (2,), 4: (1,), 7: (2,), 10: (1,), 11: (1,), 12: (2,), 13: (1,), 
              17: (1,), 18: (1,), 19: (2,), 20: (2,), 21: (1,), 23: (1, 2), 24: (2,), 25: (3,), 26: (1,),
              27: (1,), 28: (3,), 29: (2,), 30: (5,), 34: (1,), 35: (2,),
              0x140: (2, 3), 0x141: (2,), 0x142: (3, 4), 0x143: (3,), 0x144: (3, 4), 0x145: (4, 5), 0x146: (3,), 0x147: (6, 7),
-             0x148: (3,), 0x149: (1,)}
+             0x148: (3,), 0x149: (1,), 0x14B: (3, 5), 0x14C: (3,), 0x14D: (3,)}
 
 
 def op_out_temps(op):

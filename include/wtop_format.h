@@ -89,9 +89,11 @@ enum {
  * bf16 as stored in checkpoints, the residual stream, norms, gates, scores and recurrent state fp32.
  * "rows" arguments: a number, WT_ROWS_AUTO or WT_SEL_AUTO. Sizes are in elements, *_bits are fp32 bit patterns.
  *
- * OP_EMBED_ROWS     [table, ids, x_out, act_out, rows, width, vocab, dt]      x = table[id] (fp32), act = x in dt
- * OP_LINEAR         [x, w, y, rows, K, N, flags, x_col, x_stride]             y = act(x[:, x_col: x_col + K] . w^T), w bf16 [N, K];
- *                   flags: WT_LIN_*; x_stride 0 = K
+ * OP_EMBED_ROWS     [table, ids, x_out, act_out, rows, width, vocab, dt, scale_bits, act_stride, act_col]
+ *                   x = table[id] * scale (fp32), act[:, act_col: act_col + width] = x in dt; act_stride 0 = width
+ * OP_LINEAR         [x, w, y, rows, K, N, flags, x_col, x_stride, bias]       y = act(x[:, x_col: x_col + K] . w^T + bias), w bf16
+ *                   [N, K], bias fp32 [N] (0: none); flags: WT_LIN_*; x_stride 0 = K. With WT_LIN_GELU_GATE the rows of w are
+ *                   (gate, up) pairs and y [rows, N / 2] = gelu(gate) * up, the tanh form of gelu
  * OP_NORM_RESID     [y, w, x, x_out, act_out, rows, width, flags, eps_bits]   x_out = x + y / rms(y) * (b + w), w fp32;
  *                   flags: bit 0 b = 1 (weights are deviations from one) else b = 0, bit 1 act_out is bf16, bit 2 y is bf16.
  *                   x = 0: no residual; x_out / act_out = 0: not written
@@ -110,16 +112,29 @@ enum {
  *                   u = sigmoid(b)(v - S^T k), S <- S + k u^T, out = S^T q; q, k unit vectors, q * dim^-1/2
  * OP_GATED_NORM     [o, w, gate, out, rows, heads, vdim, eps_bits, flags]     out = o / rms(o) * w * sigmoid(gate) per head
  * OP_ARGMAX_ROWS    [x, out, rows, n]                                         int32 per row of fp32 x
- * OP_STATE_ADVANCE  [first, n, rows]                                          adds rows to the position counters of n states */
+ * OP_STATE_ADVANCE  [first, n, rows]                                          adds rows to the position counters of n states
+ * OP_TANH_RESID     [y, p, x, x_out, next, act_out, rows, width, flags, act_stride, act_col]
+ *                   element by element: x_out = x + t(y, p), act_out[:, act_col: act_col + width] = t(x_out, next) with
+ *                   t(z, p) = tanh(alpha z) w + b, p fp32 [alpha, 0, 0, 0 | w: width | b: width]; p, next = 0: t(z) = z;
+ *                   x = 0: no residual; x_out / act_out = 0: not written; flags: bit 1 act_out is bf16, bit 2 y is bf16
+ * OP_HEADS_APPEND   [y, norms, rope, q_out, state, rows, heads, kv_heads, dim, vdim, rot, eps_bits, y_stride, positions, dt]
+ *                   y rows = [q: heads x dim | k: kv_heads x dim | v: kv_heads x vdim | ...], each group starting at a multiple of
+ *                   8; q and k per head: / rms * norms (fp32 [q: dim | k: dim]; 0: left as they are), then the first rot components
+ *                   turned, i with i + rot / 2 (rope: fp32 [positions][rot / 2][cos, sin]). Appends [k | v] to the state, a ring:
+ *                   position p lies in row p mod (rows of the state); positions: the most the counter may reach
+ * OP_WINDOW_ATTEND  [q, y, state, out, rows, heads, kv_heads, dim, vdim, window, scale_bits, gate_col, y_stride, dt]
+ *                   softmax(q . k * scale) v over the last `window` positions up to the row's own, query head h with key head
+ *                   h / (heads / kv_heads); times sigmoid(y[:, gate_col: gate_col + heads * vdim]) unless gate_col is all ones */
 enum {
     OP_EMBED_ROWS = 0x140, OP_LINEAR, OP_NORM_RESID, OP_PICK_ROWS, OP_LATENT_APPEND, OP_LATENT_ATTEND, OP_SHORT_CONV,
-    OP_CHANNEL_DELTA, OP_GATED_NORM, OP_ARGMAX_ROWS, OP_STATE_ADVANCE, OP_ROWS_END
+    OP_CHANNEL_DELTA, OP_GATED_NORM, OP_ARGMAX_ROWS, OP_STATE_ADVANCE, OP_TANH_RESID, OP_HEADS_APPEND, OP_WINDOW_ATTEND, OP_ROWS_END
 };
 #define WT_DT_F32   0u
 #define WT_DT_BF16  1u
 #define WT_LIN_X_BF16  1u
 #define WT_LIN_Y_BF16  2u
 #define WT_LIN_RELU2   16u   /* y = max(x . w, 0)^2 */
+#define WT_LIN_GELU_GATE 32u
 #define WT_COL_ALIGN   8u    /* column groups of a joined projection start at multiples of this many elements */
 
 /* Fixed argument count per opcode (oplist_parse.h:218-251). */

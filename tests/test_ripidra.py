@@ -179,11 +179,11 @@ def test_row_ops_are_validated(cuda):
     e = RowsEmitter("float32", 64, 8, 2)
     tab = e.slot("t", lambda: np.zeros((4, 8), np.uint16))
     e.embed(tab, 4, 8)
-    e.b.add_op(OP.LINEAR, [1, S(99), 9, ROWS_AUTO, 8, 8, 0, 0, 0])
+    e.b.add_op(OP.LINEAR, [1, S(99), 9, ROWS_AUTO, 8, 8, 0, 0, 0, 0])
     assert parse_blob(cuda, e.finish())[0] == -12
     e.b.ops[-1] = (OP.LINEAR, [1, tab, 9])
     assert parse_blob(cuda, e.b.build())[0] == -11
-    e.b.ops[-1] = (0x14B, [])
+    e.b.ops[-1] = (0x14E, [])
     assert parse_blob(cuda, e.b.build())[0] == -10
 
 
@@ -284,8 +284,8 @@ def test_projection_shapes(cuda, K, N):
             def emit(e, t):
                 ws = e.slot("w", lambda: f32_to_bf16(w))
                 fl = LIN_X_BF16 if e.bf16 else 0
-                e.op(OP.LINEAR, [e.act(), ws, e.temp("y"), ROWS_AUTO, K, N, fl, 8, width])
-                e.op(OP.LINEAR, [e.act(), ws, e.temp("r"), ROWS_AUTO, K, N, fl | (LIN_Y_BF16 if e.bf16 else 0) | LIN_RELU2, 8, width])
+                e.op(OP.LINEAR, [e.act(), ws, e.temp("y"), ROWS_AUTO, K, N, fl, 8, width, 0])
+                e.op(OP.LINEAR, [e.act(), ws, e.temp("r"), ROWS_AUTO, K, N, fl | (LIN_Y_BF16 if e.bf16 else 0) | LIN_RELU2, 8, width, 0])
             eng, e, x = run_ops(cuda, emit, rows, dtype=dtype, width=width)
             want = x[:, 8:8 + K].astype(np.float64) @ w.T.astype(np.float64)
             y = eng.temp(e.temp("y"), np.float32).reshape(rows, N)
