@@ -49,7 +49,7 @@ def parse_args():
                          "3: 0.6B-shape prefill, 5: gated delta-rule layer) with its roofline and the reference's CPU time")
     ap.add_argument("--micro", default=None, choices=["gemv", "lmhead", "gemm", "swiglu", "swiglu512", "gemm1", "gemm512", "f16gemm", "headline", "gemmtiles", "attn", "attn8", "norm", "prefill", "gdn", "all"],
                     help="time single kernels (device-resident operands, graph replay) instead of the decode step")
-    ap.add_argument("--design", default=None, choices=["Ripidra"],
+    ap.add_argument("--design", default=None, choices=["Ripidra", "Supevik"],
                     help="prefill and decode of a model design at real layer sizes (random weights), beside the decoder of the same width, "
                          "feed-forward and heads with fp16 weights: tokens/s and, per launch unit, time against its roofline")
     ap.add_argument("--sizes", default="1024,2560", help="widths for --design, with commas between them")
@@ -850,9 +850,51 @@ def run_config(args):
 DESIGN_SIZES = {1024: (3072, 16), 2560: (9728, 32)}
 
 
-def design_model(width, vocab):
-    """A Ripidra model of 2 latent-attention and 2 channel-delta layers with random weights (a 1M-value block, tiled)."""
-    from gehtp_b200.checkpoint import ArrayTensors, f32_to_bf16
+def design_tensors():
+    """Random weights: function (rows, columns, scale = columns^-1/2) -> bf16 bits, tiled from a block of 1M values."""
+    from gehtp_b200.checkpoint import f32_to_bf16
+    block = np.random.default_rng(9).standard_normal(1 << 20, dtype=np.float32)
+
+    def mat(n, k, scale=None):
+        b = f32_to_bf16(block * np.float32(k ** -0.5 if scale is None else scale))
+        return np.resize(b, (n, k)) if k else np.resize(b, n)
+    return mat
+
+
+def design_model(design, width, vocab):
+    return {"Ripidra": ripidra_model, "Supevik": supevik_model}[design](width, vocab)
+
+
+def supevik_model(width, vocab):
+    """A Supevik model of 3 layers, the middle one run twice over the whole context, the others over windows of 1024."""
+    from gehtp_b200.checkpoint import ArrayTensors
+    from gehtp_b200.registry import Model
+    ff, H = DESIGN_SIZES[width]
+    G, mat = 8, design_tensors()
+    rot = dict(base=1e6, dims=128, scaling=dict(factor=4.0, fast=32.0, slow=1.0, original=2048))
+    layers = [dict(type="attention", mlp=dict(kind="dense", ff=ff),
+                   mixer=dict(heads=H, kv_heads=G, dim=128, vdim=128, mask=dict(size=n), rot=rot, scale=128 ** -0.5)) for n in (1024, 8192, 1024)]
+    cfg = dict(architecture="Supevik", vocab=vocab, width=width, norm=dict(eps=1e-6), embedding=dict(scale=4.0), layers=layers,
+               loop=dict(start=1, stop=2, times=2))
+    t = {"embed": mat(vocab, width, 1.0), "head": mat(vocab, width), "loop.in": mat(width, 2 * width)}
+
+    def norm(name):
+        t[name], t[name + ".b"], t[name + ".alpha"] = mat(width, 0, 1.0), mat(width, 0, 0.1), np.full(1, 0.5, np.float32)
+    norm("final.norm")
+    for i in range(3):
+        p, q = "l%d." % i, "l%d.mix." % i
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            norm(p + n)
+        t.update({q + "q": mat(H * 128, width), q + "k": mat(G * 128, width), q + "v": mat(G * 128, width), q + "g": mat(H * 128, width),
+                  q + "o": mat(width, H * 128), q + "q.b": mat(H * 128, 0, 0.1), q + "k.b": mat(G * 128, 0, 0.1), q + "v.b": mat(G * 128, 0, 0.1),
+                  q + "q.norm": mat(128, 0, 1.0), q + "k.norm": mat(128, 0, 1.0),
+                  p + "mlp.gate": mat(ff, width), p + "mlp.up": mat(ff, width), p + "mlp.down": mat(width, ff)})
+    return Model(cfg, ArrayTensors(t))
+
+
+def ripidra_model(width, vocab):
+    """A Ripidra model of 2 latent-attention and 2 channel-delta layers with random weights."""
+    from gehtp_b200.checkpoint import ArrayTensors
     from gehtp_b200.registry import Model
     ff, H = DESIGN_SIZES[width]
     lat = dict(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=512, rot=dict(base=1e6, dims=64), scale=192 ** -0.5)
@@ -860,11 +902,7 @@ def design_model(width, vocab):
     kinds = [("channel_delta", dlt), ("latent_attention", lat)] * 2
     cfg = dict(architecture="Ripidra", vocab=vocab, width=width, norm=dict(eps=1e-6),
                layers=[dict(type=k, mixer=m, mlp=dict(kind="dense", ff=ff)) for k, m in kinds])
-    block = np.random.default_rng(9).standard_normal(1 << 20, dtype=np.float32)
-
-    def mat(n, k, scale=None):
-        b = f32_to_bf16(block * np.float32(k ** -0.5 if scale is None else scale))
-        return np.resize(b, (n, k)) if k else np.resize(b, n)
+    mat = design_tensors()
     t = {"embed": mat(vocab, width, 1.0), "final.norm": mat(width, 0, 0.1)}
     for i, (k, m) in enumerate(kinds):
         p = "l%d." % i
@@ -944,7 +982,7 @@ def run_design(args, width):
                       "tok_s": round(tokens / ms * 1e3, 1), "units": un, "clocks": clocks, "l2": "overwritten before every timed step"})
 
     # ---- the design
-    s = Session(design_model(width, V), max_tokens=CTX, max_rows=S_, max_sel=16)
+    s = Session(design_model(args.design, width, V), max_tokens=CTX, max_rows=S_, max_sel=16)
     eng, man = s.engine, s.man
     rng = np.random.default_rng(5)
 
@@ -970,6 +1008,28 @@ def run_design(args, width):
             return "other", 0, 0
         return f
 
+    def work_window(rows, past):
+        fused = {i for i in range(eng.blob.n_ops - 1) if eng.blob.ops[i].opcode == OP.LINEAR and eng.blob.ops[i + 1].opcode == OP.TANH_RESID}
+
+        def f(i, op):
+            a = list(op.args)
+            if op.opcode == OP.LINEAR:
+                r, k, c = 1 if a[3] == SEL_AUTO else rows, a[4], a[5]
+                if i in fused:
+                    return "linear %dx%d + norms, residual" % (k, c), 2 * k * c + r * (2 * k + 10 * c), 2.0 * r * k * c
+                if a[6] & 32:
+                    return "linear %dx%d, gated gelu" % (k, c), 2 * k * c + r * (2 * k + c), 2.0 * r * k * c
+                return "linear %dx%d" % (k, c), 2 * k * c + r * (2 * k + (2 if a[6] & 2 else 4) * c), 2.0 * r * k * c
+            if op.opcode in (OP.HEADS_APPEND, OP.WINDOW_ATTEND):
+                n = next(eng.blob.ops[j].args[9] for j in (i, i + 1) if eng.blob.ops[j].opcode == OP.WINDOW_ATTEND)
+                io = rows * (3 * H + 2 * 8) * 128 * 2
+                pairs = sum(min(past + r + 1, n) for r in range(rows))
+                return "append + attention, window %d" % n, io + (min(past, n) * 8 * 256 * 2 if rows == 1 else rows * 8 * 512), 4.0 * H * 128 * pairs
+            if op.opcode == OP.TANH_RESID:
+                return "norm", rows * width * 6, 0
+            return "other", 0, 0
+        return f
+
     def phase(rows, ctx, name):
         face = np.zeros(man["max_rows"] + man["max_sel"], np.int32)
         face[:rows] = rng.integers(0, V, rows)
@@ -982,14 +1042,14 @@ def run_design(args, width):
         eng.set_rows(rows, 1)
 
         def rewind():
-            for i in range(2):
+            for i in range({"Ripidra": 2, "Supevik": 4}[args.design]):
                 assert lib.gehtp_cuda_state_set_count(i, ctx) == 0
 
         def step():
             assert lib.gehtp_cuda_run_dev(ctypes.byref(eng.blob), dface.data_ptr(), out.data_ptr(), man["token_temp"], err, 256) == 0, err.value
         ms = timed(step, rewind)
         rewind()
-        un = units(eng, face, man["token_temp"], work_rows(rows, ctx))
+        un = units(eng, face, man["token_temp"], {"Ripidra": work_rows, "Supevik": work_window}[args.design](rows, ctx))
         add(args.design, name, ms, rows, un)
 
     sampler = ClockSampler(0)
@@ -1049,6 +1109,8 @@ def run_design(args, width):
     rewind()
     add(cfg.name, "decode ctx %d" % (CTX - 64), ms, 1, units(eng, face, man["token_temp"], work_fixed(1, CTX)))
     eng.shutdown()
+    if args.design != "Ripidra":
+        return lines
     # ---- the delta rule of the gated-delta layer (config 5) at the same heads: chunks of 64 tokens, convolution over 3 H 128 channels
     buf, man = build_gdn_runlist(S_, width, 3 * H * 128, 4, H, 128, 64)
     eng = Engine(lib, buf)

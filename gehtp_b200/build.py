@@ -40,6 +40,7 @@ UNITS = {
     "latent_prefill.cu": [],
     "window_attn.cu": [],
     "window_prefill.cu": [],
+    "window_attn_sm100.cu": [],
     "channel_delta.cu": [],
     "tp.cu": [],
     "tp_p2p.cu": [],

@@ -83,6 +83,9 @@ template <> struct InOf<EpiF16> {
     static constexpr uint32_t IDESC = 0;
 };
 
+template <class E> struct Heavy { static constexpr bool value = false; };
+template <class A> struct Heavy<EpiTanh<A>> { static constexpr bool value = true; };
+
 // fp16 outputs: rows ldy elements apart (the SPLIT form writes N columns of a row of N_full).
 template <int MH, int BN, class E>
 __global__ void __launch_bounds__(NTHREADS, 1)
@@ -102,8 +105,8 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t KG = IO::EDGE ? (K + BK - 1) / BK : K / BK;
     const uint32_t m_tiles = (M + 128 * MH - 1) / (128 * MH), tiles = m_tiles * (IO::EDGE ? (N + BN - 1) / BN : N / BN);
-    // Split K (S > 1): a work item is (tile, run of K/64/S k blocks), item = run * tiles + tile; a run leaves its fp32
-    // partial sums in part[run][row][N] and f16_splitk_reduce_kernel adds the runs in order.
+    // Split K (S > 1): a work item is (tile, run of K/64/S k blocks), item = run * tiles + tile. With `part` a run leaves its
+    // fp32 sums in part[run][row][N]; f16_splitk_reduce_kernel adds the runs in order and applies the epilogue.
     const uint32_t items = tiles * S, KGS = KG / S;
 
     if (threadIdx.x == 0) {
@@ -203,7 +206,7 @@ f16_gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
                         : "r"(taddr));
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                     const uint32_t n = n0 + c * 32;
-                    if (m < M && S > 1) {
+                    if (m < M && part) {
                         // rows of the partial sums are N rounded up to 4 floats apart
                         const uint32_t np = IO::EDGE ? (N + 3) & ~3u : N;
                         uint4* dst = (uint4*)(part + ((size_t)run * M + m) * np + n);
@@ -287,11 +290,13 @@ bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w,
             unsigned int* status, int sms) {
     using C = FCfg<MH, BN>;
     using IO = InOf<E>;
+    // an epilogue that is too much for four warps goes to the reduction kernel even of a single run
+    using G = typename std::conditional<Heavy<E>::value, EpiPlain<false, false>, E>::type;
     CUtensorMap ta, tw;
     if (!make_map(&ta, IO::MAP, a, M, K, lda, 128) || !make_map(&tw, IO::MAP, w, N, K, K, BN)) return false;
     const size_t smem = 1024 + (size_t)C::STAGES * (C::A_BYTES + C::B_BYTES) + sizeof(FBarriers) + 16;
     static int have[64] = {};
-    if (!ensure_dyn_smem(f16_gemm_sm100_kernel<MH, BN, E>, smem, have)) return false;
+    if (!ensure_dyn_smem(f16_gemm_sm100_kernel<MH, BN, G>, smem, have)) return false;
     const uint32_t tiles = ((M + 128 * MH - 1) / (128 * MH)) * ((N + BN - 1) / BN), KG = (K + BK - 1) / BK;
     const uint32_t np = (N + 3) & ~3u;
     // Split K while the tiles alone leave SMs idle (same rule as the W4A16 GEMM): the divisor of K/64 that makes
@@ -307,18 +312,21 @@ bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w,
         }
     }
     float* part = nullptr;
-    if (S > 1) {
+    if (S > 1 || Heavy<E>::value) {
         SplitScratch* ss = split_scratch(st, (size_t)S * M * np * sizeof(float));
         if (ss) part = ss->part; else S = 1;
     }
+    G direct{};
+    if constexpr (!Heavy<E>::value) direct = epi;
+    else if (!part) return false;
     const uint32_t items = tiles * S;
     const uint32_t grid = items < (uint32_t)sms ? items : (uint32_t)sms;
-    if (launch_pdl(f16_gemm_sm100_kernel<MH, BN, E>, dim3(grid), dim3(NTHREADS), smem, st, ta, tw, epi, M, K, N, status, S, part) != cudaSuccess) {
+    if (launch_pdl(f16_gemm_sm100_kernel<MH, BN, G>, dim3(grid), dim3(NTHREADS), smem, st, ta, tw, direct, M, K, N, status, S, part) != cudaSuccess) {
         cudaGetLastError();
         return false;
     }
     g_launches++;
-    if (S > 1) {
+    if (part) {
         const size_t quads = (size_t)M * np / 4;
         uint32_t rg = (uint32_t)((quads + 255) / 256);
         if (rg > (uint32_t)sms * 8) rg = (uint32_t)sms * 8;
@@ -473,6 +481,10 @@ bool launch_tiles(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16
         if (sms <= 0) sms = 148;
     }
     const uint32_t t256 = ((M + 255) / 256) * ((N + 255) / 256), t128 = ((M + 255) / 256) * ((N + 127) / 128);
+    // row-count projections: the wider tile where its rounds over the SMs are not worth more than those of the narrow one
+    // (0.55 of its time, and an epilogue that overlaps the next tile's products)
+    const uint32_t r256 = (t256 + sms - 1) / sms, r128 = (t128 + sms - 1) / sms;
+    if (InOf<E>::EDGE && M > 128 && t128 >= (uint32_t)sms && 11 * r128 < 20 * r256) return launch<2, 128, E>(st, a, lda, w, epi, M, K, N, status, sms);
     if ((InOf<E>::EDGE || N % 256 == 0) && M > 128 && t256 >= (uint32_t)sms) return launch<2, 256, E>(st, a, lda, w, epi, M, K, N, status, sms);
     if (M > 128 && t128 >= (uint32_t)sms) return launch<2, 128, E>(st, a, lda, w, epi, M, K, N, status, sms);
     return launch<1, 128, E>(st, a, lda, w, epi, M, K, N, status, sms);

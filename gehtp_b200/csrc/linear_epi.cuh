@@ -5,6 +5,7 @@
 //   chunk(m, n, f, N)       columns n .. n + 31 (n a multiple of 32)
 // Columns at or past N are left out.
 #pragma once
+#include <type_traits>
 #include "rows_common.cuh"
 
 namespace gehtp {
@@ -40,6 +41,17 @@ struct EpiPlain {
         for (uint32_t k = 0; k < 4; k++) if (n + k < N) one(m, n + k, v[k]);
     }
     __device__ __forceinline__ void chunk(uint32_t m, uint32_t n, const float (&f)[32], uint32_t N) const {
+        if (YB && !RELU2 && bias && n + 32 <= N && ((uintptr_t)(bias + n) & 15u) == 0 && (((uintptr_t)y + ((size_t)m * ldy + n) * 2) & 15u) == 0) {
+            uint4* d = (uint4*)((uint16_t*)y + (size_t)m * ldy + n);
+#pragma unroll
+            for (uint32_t q = 0; q < 4; q++) {
+                const float4 a = __ldg((const float4*)(bias + n) + 2 * q), b = __ldg((const float4*)(bias + n) + 2 * q + 1);
+                const float* v = f + 8 * q;
+                d[q] = make_uint4(pack_bf2(v[0] + a.x, v[1] + a.y), pack_bf2(v[2] + a.z, v[3] + a.w), pack_bf2(v[4] + b.x, v[5] + b.y),
+                                  pack_bf2(v[6] + b.z, v[7] + b.w));
+            }
+            return;
+        }
 #pragma unroll
         for (uint32_t q = 0; q < 4; q++) {
             const uint32_t c = n + 8 * q;
@@ -58,6 +70,17 @@ struct EpiPlain {
     }
 };
 
+// tanh and 1 / (1 + e^-z) by output type: the library functions where fp32 comes out; beside bf16 outputs forms on the
+// hardware exponential and reciprocal, whose absolute error stays within a few 2^-23.
+template <class A> struct Curve {
+    static __device__ __forceinline__ float tanh_(float z) { return tanhf(z); }
+    static __device__ __forceinline__ float sigmoid(float z) { return sigmoid_f(z); }
+};
+template <> struct Curve<ActBf16> {
+    static __device__ __forceinline__ float tanh_(float z) { return fmaf(-2.0f, sigmoid_fast(-2.0f * z), 1.0f); }
+    static __device__ __forceinline__ float sigmoid(float z) { return sigmoid_fast(z); }
+};
+
 // Columns are (gate, up) pairs: y[m][n / 2] = gelu(gate) * up. The tanh form of gelu, z (1 + tanh u) / 2, is z sigmoid(2u).
 template <bool YB>
 struct EpiGelu {
@@ -65,7 +88,7 @@ struct EpiGelu {
     uint32_t ldy;
     static __device__ __forceinline__ float val(float z, float up) {
         const float u = 0.79788456080286535588f * fmaf(0.044715f * z * z, z, z);      // sqrt(2 / pi)
-        return z / (1.0f + expf(-2.0f * u)) * up;
+        return z * Curve<typename std::conditional<YB, ActBf16, ActF32>::type>::sigmoid(2.0f * u) * up;
     }
     __device__ __forceinline__ void pair(uint32_t m, uint32_t n, float v0, float v1, uint32_t N) const {
         if (n + 1 >= N) return;
@@ -98,8 +121,9 @@ struct EpiGelu {
 };
 
 // t(z, p) = tanh(alpha z) w + b of one column; p = [alpha, 0, 0, 0 | w: width | b: width], none: z
+template <class A>
 __device__ __forceinline__ float tanh_norm(const float* p, uint32_t width, uint32_t n, float z) {
-    return p ? fmaf(tanhf(__ldg(p) * z), __ldg(p + 4 + n), __ldg(p + 4 + width + n)) : z;
+    return p ? fmaf(Curve<A>::tanh_(__ldg(p) * z), __ldg(p + 4 + n), __ldg(p + 4 + width + n)) : z;
 }
 
 // x_out = x + t(v, p), act = t(x_out, next): the element-wise norm behind a sublayer, the residual sum and the norm in
@@ -113,9 +137,9 @@ struct EpiTanh {
     bool vec;                          // rows of 16-byte quads (fp32) and 8- or 16-byte quads (act)
     __device__ __forceinline__ void one(uint32_t m, uint32_t n, float v) const {
         const size_t i = (size_t)m * width + n;
-        const float s = (x ? __ldcg(x + i) : 0.0f) + tanh_norm(p, width, n, v);
+        const float s = (x ? __ldcg(x + i) : 0.0f) + tanh_norm<A>(p, width, n, v);
         if (x_out) x_out[i] = s;
-        if (act) A::st(act + (size_t)m * act_ld + n, tanh_norm(next, width, n, s));
+        if (act) A::st(act + (size_t)m * act_ld + n, tanh_norm<A>(next, width, n, s));
     }
     __device__ __forceinline__ void pair(uint32_t m, uint32_t n, float v0, float v1, uint32_t N) const {
         if (n < N) one(m, n, v0);
@@ -126,7 +150,8 @@ struct EpiTanh {
         if (!q) return z;
         const float a = __ldg(q);
         const float4 w = __ldg((const float4*)(q + 4 + n)), b = __ldg((const float4*)(q + 4 + width + n));
-        return make_float4(fmaf(tanhf(a * z.x), w.x, b.x), fmaf(tanhf(a * z.y), w.y, b.y), fmaf(tanhf(a * z.z), w.z, b.z), fmaf(tanhf(a * z.w), w.w, b.w));
+        return make_float4(fmaf(Curve<A>::tanh_(a * z.x), w.x, b.x), fmaf(Curve<A>::tanh_(a * z.y), w.y, b.y),
+                           fmaf(Curve<A>::tanh_(a * z.z), w.z, b.z), fmaf(Curve<A>::tanh_(a * z.w), w.w, b.w));
     }
     __device__ __forceinline__ float4 res4(uint32_t m, uint32_t n) const {
         return x ? __ldcg((const float4*)(x + (size_t)m * width + n)) : make_float4(0.f, 0.f, 0.f, 0.f);

@@ -227,7 +227,7 @@ void plan_rows_op(Planner& P, const wt_op& op, PlanOp& p) {
             p.pos_append_state = si;
             if (P.build) p.launch = [=](cudaStream_t st) { k_heads_append(st, w, rows_of(rows)); };
         } else {
-            w.window = a[9]; w.scale = from_bits(a[10]); w.gate_col = a[11];
+            w.window = a[9] < 0x40000000u ? a[9] : 0x40000000u; w.scale = from_bits(a[10]); w.gate_col = a[11];
             const bool gate = w.gate_col != 0xFFFFFFFFu;
             if (!w.window) FAIL("window of no positions");
             // a run's rows are appended before they attend: the ring holds them and the windows behind the first of them,

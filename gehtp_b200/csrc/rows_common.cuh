@@ -25,6 +25,8 @@ struct ActBf16 {
 };
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+// the same on the hardware exponential and reciprocal, within a few 2^-23 of it: beside outputs that are rounded to bf16
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(fminf(-z, 80.0f))); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 
 // sum over the whole block; `part` holds one float per warp. Every thread gets the sum.

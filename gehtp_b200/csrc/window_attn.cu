@@ -24,6 +24,9 @@ __device__ __forceinline__ void head_row(const typename A::T* src, uint32_t dim,
                                          float* buf, F&& out) {
     const uint32_t lane = threadIdx.x & 31, half = rot / 2;
     float ss = 0.0f;
+    float2 early[2];                               // constants, on their way while the row is summed
+#pragma unroll
+    for (int u = 0; u < 2; u++) early[u] = lane + 32 * u < half ? __ldg(rope + lane + 32 * u) : make_float2(0.f, 0.f);
     if (sizeof(typename A::T) == 2 && ((dim | (uint32_t)((uintptr_t)src >> 1)) & 1u) == 0) {
         for (uint32_t i = 2 * lane; i < dim; i += 64) {
             const uint32_t w = __ldcg((const uint32_t*)(src + i));
@@ -43,7 +46,7 @@ __device__ __forceinline__ void head_row(const typename A::T* src, uint32_t dim,
     __syncwarp();
     auto val = [&](uint32_t i) { return nw ? buf[i] * inv * __ldg(nw + i) : buf[i]; };
     for (uint32_t i = lane; i < half; i += 32) {
-        const float2 cs = __ldg(rope + i);
+        const float2 cs = i < 32 ? early[0] : i < 64 ? early[1] : __ldg(rope + i);
         const float u = val(i), v = val(i + half);
         buf[i] = u * cs.x - v * cs.y;
         buf[i + half] = v * cs.x + u * cs.y;
@@ -63,31 +66,111 @@ __device__ __forceinline__ void put_pair(typename A::T* dst, uint32_t i, uint32_
     }
 }
 
-// one CTA per row, a warp per head; dynamic shared memory: [8][dim + 1] floats
+// a warp per row and head (queries, then keys, then values); dynamic shared memory: [8][dim + 1] floats
 template <class A>
 __global__ void __launch_bounds__(256)
 heads_append_kernel(const WindowArgs a) {
     extern __shared__ float sm[];
     typedef typename A::T T;
     pdl_release();
+    const uint32_t r = blockIdx.x, pos = *(volatile const uint32_t*)a.counter + r, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t h = blockIdx.y * 8 + warp;
     pdl_wait();
-    const uint32_t r = blockIdx.x, pos = *a.counter + r, warp = threadIdx.x >> 5;
-    if (pos >= a.positions) return;                 // the host has checked the room
-    float* buf = sm + warp * (a.dim + 1);
+    if (pos >= a.positions || h >= a.heads + 2 * a.kv_heads) return;            // the host has checked the room
     const T* y = (const T*)a.y + (size_t)r * a.y_cols;
-    const float2* rope = (const float2*)a.rope + (size_t)pos * (a.rot / 2);
     T* dst = (T*)a.state + (size_t)(pos % a.ring) * a.row();
-    T* q = (T*)a.q + (size_t)r * a.heads * a.dim;
-    for (uint32_t h = warp; h < a.heads + a.kv_heads; h += 8) {
-        const bool key = h >= a.heads;
-        const uint32_t k = h - a.heads;
-        T* to = key ? dst + k * a.dim : q + h * a.dim;
-        head_row<A>(key ? y + a.col_k() + k * a.dim : y + h * a.dim, a.dim, a.norms ? a.norms + (key ? a.dim : 0) : nullptr, rope, a.rot, a.eps, buf,
-                    [&](uint32_t i, float u, float v) { put_pair<A>(to, i, a.dim, u, v); });
+    if (h >= a.heads + a.kv_heads) {
+        const uint32_t g = h - a.heads - a.kv_heads;
+        const T* v = y + a.col_v() + g * a.vdim;
+        T* to = dst + a.kv_heads * a.dim + g * a.vdim;
+        if (a.vdim % 8 == 0 && (((uintptr_t)v | (uintptr_t)to) & 15u) == 0)
+            for (uint32_t i = lane; i < a.vdim * sizeof(T) / 16; i += 32) ((uint4*)to)[i] = __ldcg((const uint4*)v + i);
+        else
+            for (uint32_t i = lane; i < a.vdim; i += 32) to[i] = __ldcg(v + i);
+        return;
     }
-    const T* v = y + a.col_v();
-    T* dv = dst + a.kv_heads * a.dim;
-    for (uint32_t i = threadIdx.x; i < a.kv_heads * a.vdim; i += 256) dv[i] = __ldcg(v + i);
+    const bool key = h >= a.heads;
+    const uint32_t k = h - a.heads;
+    T* to = key ? dst + k * a.dim : (T*)a.q + ((size_t)r * a.heads + h) * a.dim;
+    head_row<A>(key ? y + a.col_k() + k * a.dim : y + h * a.dim, a.dim, a.norms ? a.norms + (key ? a.dim : 0) : nullptr,
+                (const float2*)a.rope + (size_t)pos * (a.rot / 2), a.rot, a.eps, sm + warp * (a.dim + 1),
+                [&](uint32_t i, float u, float v) { put_pair<A>(to, i, a.dim, u, v); });
+}
+
+// Eight neighbouring components of one head of LP * 8, a lane each: norm, then the first `rot` components turned; rotation
+// partners lie rot / 16 lanes apart. The constants are fetched on construction, ahead of the data.
+template <int LP>
+struct HeadVec {
+    float nw[8], cs[8], sn[8];
+    uint32_t mate;
+    bool norm;
+    __device__ __forceinline__ HeadVec(bool live, uint32_t c, const float* norms, const float* rope, uint32_t pos, uint32_t rot) {
+        const uint32_t hl = rot / 16, lane = threadIdx.x & 31;
+        norm = norms != nullptr;
+        mate = c < hl ? lane + hl : c < 2 * hl ? lane - hl : lane;
+#pragma unroll
+        for (int i = 0; i < 8; i++) { nw[i] = 1.0f; cs[i] = 1.0f; sn[i] = 0.0f; }
+        if (!live) return;
+        if (norms) {
+            const float4* n = (const float4*)(norms + c * 8);
+            const float4 n0 = __ldg(n), n1 = __ldg(n + 1);
+            nw[0] = n0.x; nw[1] = n0.y; nw[2] = n0.z; nw[3] = n0.w; nw[4] = n1.x; nw[5] = n1.y; nw[6] = n1.z; nw[7] = n1.w;
+        }
+        if (c < 2 * hl) {                          // the second half of the pairs turns with the other sign
+            const float4* t = (const float4*)((const float2*)rope + (size_t)pos * (rot / 2) + (c < hl ? c : c - hl) * 8);
+            const float f = c < hl ? -1.0f : 1.0f;
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const float4 q = __ldg(t + i);
+                cs[2 * i] = q.x; sn[2 * i] = f * q.y; cs[2 * i + 1] = q.z; sn[2 * i + 1] = f * q.w;
+            }
+        }
+    }
+    // every lane of the warp takes part
+    __device__ __forceinline__ uint4 turn(uint4 w, float eps) const {
+        const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
+        float x[8], o[8], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 4; i++) { x[2 * i] = __uint_as_float(ww[i] << 16); x[2 * i + 1] = __uint_as_float(ww[i] & 0xffff0000u); }
+#pragma unroll
+        for (int i = 0; i < 8; i++) ss = fmaf(x[i], x[i], ss);
+#pragma unroll
+        for (int d = LP / 2; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+        const float inv = norm ? 1.0f / sqrtf(ss / (float)(LP * 8) + eps) : 1.0f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            x[i] = x[i] * inv * nw[i];
+            o[i] = fmaf(__shfl_sync(0xffffffffu, x[i], mate), sn[i], x[i] * cs[i]);
+        }
+        return make_uint4(pack_bf2(o[0], o[1]), pack_bf2(o[2], o[3]), pack_bf2(o[4], o[5]), pack_bf2(o[6], o[7]));
+    }
+};
+
+// sizes and alignment the 8-component form takes
+bool head_vec(const WindowArgs& a) {
+    const uint32_t lp = a.dim / 8;
+    const uintptr_t al = (uintptr_t)a.y | (uintptr_t)a.q | (uintptr_t)a.state | (uintptr_t)a.norms | (uintptr_t)a.rope;
+    return a.bf16 && a.dim % 8 == 0 && (lp == 8 || lp == 16 || lp == 32) && a.rot % 16 == 0 && a.vdim % 8 == 0 && a.y_cols % 8 == 0 && (al & 15u) == 0;
+}
+
+// heads_append_kernel for such heads: a thread per 8 components; grid (rows, items / 256)
+template <int LP>
+__global__ void __launch_bounds__(256)
+heads_append_vec_kernel(const WindowArgs a) {
+    pdl_release();
+    const uint32_t r = blockIdx.x, pos = *(volatile const uint32_t*)a.counter + r, item = blockIdx.y * 256 + threadIdx.x;
+    const uint32_t nq = (a.heads + a.kv_heads) * LP, nv = a.kv_heads * (a.vdim / 8), h = item / LP, c = item % LP;
+    const bool head = item < nq, key = h >= a.heads, live = item < nq + nv && pos < a.positions;
+    const uint32_t v = item - nq;
+    const uint16_t* y = (const uint16_t*)a.y + (size_t)r * a.y_cols;
+    uint16_t* dst = (uint16_t*)a.state + (size_t)(pos % a.ring) * a.row();
+    const uint16_t* src = !head ? y + a.col_v() + v * 8 : key ? y + a.col_k() + (h - a.heads) * LP * 8 + c * 8 : y + h * LP * 8 + c * 8;
+    uint16_t* to = !head ? dst + a.kv_heads * LP * 8 + v * 8 : key ? dst + (h - a.heads) * LP * 8 + c * 8 : (uint16_t*)a.q + ((size_t)r * a.heads + h) * LP * 8 + c * 8;
+    const HeadVec<LP> hv(live && head, c, a.norms ? a.norms + (key ? LP * 8 : 0) : nullptr, a.rope, pos, a.rot);
+    pdl_wait();
+    const uint4 w = live ? __ldcg((const uint4*)src) : make_uint4(0, 0, 0, 0);
+    const uint4 o = hv.turn(w, a.eps);
+    if (live) *(uint4*)to = head ? o : w;
 }
 
 // Attention of one (head, row): running softmax over blocks of 128 keys. Dynamic shared memory: [dim] query, [vdim] sums.
@@ -145,10 +228,10 @@ window_exact_kernel(const WindowArgs a) {
 // 16-row MMA tile. APPEND: the row's own key and value come from the projection and are stored to the ring by one CTA.
 // Positions below the counter were written by earlier runs and the counter moves at the end of a run only: tiles of such
 // positions are requested before the dependency wait.
-constexpr uint32_t SP = 16, SW = 8;               // positions per tile, warps
-template <int VT, bool VEC, bool APPEND>
+constexpr uint32_t SP = 16, SW = 8, MAXC = 16;    // positions per tile, warps, CTAs of a cluster at most
+template <int VT, bool VEC, bool APPEND, int LP>
 __global__ void __launch_bounds__(256)
-window_step_kernel(const WindowArgs a) {
+window_step_kernel(const WindowArgs a, uint32_t stages) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float wm[SW][16], wl[SW][16], cm[16], cl[16];
     cooperative_groups::cluster_group cluster = cooperative_groups::this_cluster();
@@ -156,7 +239,7 @@ window_step_kernel(const WindowArgs a) {
     uint16_t* sq = (uint16_t*)smem;                               // [16][rk]
     uint16_t* snew = sq + 16 * rk;                                // [dp + vp]: this row's key and value
     float* scr = (float*)(snew + dp + vp);                        // [SW][dim + 2]
-    uint16_t* tiles = (uint16_t*)(scr + SW * (((a.dim + 2) + 3u) & ~3u));
+    uint16_t* tiles = (uint16_t*)(scr + (LP ? 0 : SW * (((a.dim + 2) + 3u) & ~3u)));
     const uint32_t tile_el = SP * (rk + rv);
     float* acc = (float*)tiles;                                   // [SW][16][vp], after the last tile
     pdl_release();
@@ -167,7 +250,7 @@ window_step_kernel(const WindowArgs a) {
     const uint32_t first = pos + 1 > a.window ? pos + 1 - a.window : 0;
     const uint32_t known = APPEND ? pos : pos + 1;                // positions whose rows are in the ring for this row
     const uint32_t t_end = pos / SP + 1, stride = C * SW;
-    uint16_t* my = tiles + warp * 2 * tile_el;
+    uint16_t* my = tiles + warp * stages * tile_el;
     const uint16_t *keys = (const uint16_t*)a.state + g * a.dim, *vals = (const uint16_t*)a.state + a.kv_heads * a.dim + g * a.vdim;
     auto fetch = [&](uint32_t t, uint32_t stage) {
         if (t < t_end) {
@@ -194,40 +277,54 @@ window_step_kernel(const WindowArgs a) {
     };
     // columns no copy writes: padding of a head to 16
     if (dp > a.dim || vp > a.vdim) {
-        for (uint32_t i = lane; i < 2 * SP * (dp - a.dim); i += 32) {
+        for (uint32_t i = lane; i < stages * SP * (dp - a.dim); i += 32) {
             const uint32_t p = i / (dp - a.dim);
             my[(p / SP) * tile_el + (p % SP) * rk + a.dim + i % (dp - a.dim)] = 0;
         }
-        for (uint32_t i = lane; i < 2 * SP * (vp - a.vdim); i += 32) {
+        for (uint32_t i = lane; i < stages * SP * (vp - a.vdim); i += 32) {
             const uint32_t p = i / (vp - a.vdim);
             my[(p / SP) * tile_el + SP * rk + (p % SP) * rv + a.vdim + i % (vp - a.vdim)] = 0;
         }
     }
+    // the first tiles, one a stage; those of earlier runs' positions ahead of the dependency wait
     const uint32_t t0 = first / SP + blockIdx.x * SW + warp;
-    const bool early0 = VEC && (t0 + 1) * SP <= past, early1 = VEC && (t0 + stride + 1) * SP <= past;
-    if (early0) fetch(t0, 0);
-    if (early0 && early1) fetch(t0 + stride, 1);
+    uint32_t ahead = 0;
+    if (VEC) for (; ahead < stages && (t0 + ahead * stride + 1) * SP <= past; ahead++) fetch(t0 + ahead * stride, ahead);
+    // LP: the heads of this group, then its key, LP lanes each; what needs no projection is fetched ahead as well
+    constexpr int LQ = LP ? LP : 8;
+    const uint32_t item_h = tid / LQ, item_c = tid % LQ;
+    const HeadVec<LQ> hv(LP && APPEND && item_h <= nh, item_c, a.norms ? a.norms + (item_h == nh ? a.dim : 0) : nullptr, a.rope, pos, a.rot);
     pdl_wait();
-    for (uint32_t i = tid; i < 16 * rk; i += 256) sq[i] = 0;
-    __syncthreads();
+    if (nh < 16) for (uint32_t i = nh * rk + tid; i < 16 * rk; i += 256) sq[i] = 0;
+    if (dp > a.dim) for (uint32_t i = tid; i < nh * (dp - a.dim); i += 256) sq[(i / (dp - a.dim)) * rk + a.dim + i % (dp - a.dim)] = 0;
     if (APPEND) {
-        // heads of this group, then the key, by warps; the value by whichever threads come
         const uint16_t* y = (const uint16_t*)a.y + (size_t)r * a.y_cols;
-        const float2* rope = (const float2*)a.rope + (size_t)pos * (a.rot / 2);
-        float* buf = scr + warp * (((a.dim + 2) + 3u) & ~3u);
-        for (uint32_t h = warp; h <= nh; h += SW) {
-            const bool key = h == nh;
-            uint16_t* to = key ? snew : sq + h * rk;
-            head_row<ActBf16>(key ? y + a.col_k() + g * a.dim : y + (h0 + h) * a.dim, a.dim, a.norms ? a.norms + (key ? a.dim : 0) : nullptr,
-                              rope, a.rot, a.eps, buf, [&](uint32_t i, float u, float v) { put_pair<ActBf16>(to, i, a.dim, u, v); });
+        if (LP) {
+            // 256 threads take 256 / LP heads at a time; the constants of the second round on are not fetched ahead
+            for (uint32_t h = item_h; h - item_h <= nh; h += 256 / LQ) {
+                const bool live = h <= nh, key = h == nh;
+                const uint4 w = live ? __ldcg((const uint4*)(y + (key ? a.col_k() + g * a.dim : (h0 + h) * a.dim) + item_c * 8)) : make_uint4(0, 0, 0, 0);
+                uint4 o;
+                if (h == item_h) o = hv.turn(w, a.eps);
+                else o = HeadVec<LQ>(live, item_c, a.norms ? a.norms + (key ? a.dim : 0) : nullptr, a.rope, pos, a.rot).turn(w, a.eps);
+                if (live) *(uint4*)((key ? snew : sq + h * rk) + item_c * 8) = o;
+            }
+        } else {
+            const float2* rope = (const float2*)a.rope + (size_t)pos * (a.rot / 2);
+            float* buf = scr + warp * (((a.dim + 2) + 3u) & ~3u);
+            for (uint32_t h = warp; h <= nh; h += SW) {
+                const bool key = h == nh;
+                uint16_t* to = key ? snew : sq + h * rk;
+                head_row<ActBf16>(key ? y + a.col_k() + g * a.dim : y + (h0 + h) * a.dim, a.dim, a.norms ? a.norms + (key ? a.dim : 0) : nullptr,
+                                  rope, a.rot, a.eps, buf, [&](uint32_t i, float u, float v) { put_pair<ActBf16>(to, i, a.dim, u, v); });
+            }
         }
         for (uint32_t i = tid; i < a.vdim; i += 256) snew[dp + i] = __ldcg(y + a.col_v() + g * a.vdim + i);
     } else {
         const uint16_t* q = (const uint16_t*)a.q + ((size_t)r * a.heads + h0) * a.dim;
         for (uint32_t i = tid; i < nh * a.dim; i += 256) sq[(i / a.dim) * rk + i % a.dim] = __ldcg(q + i);
     }
-    if (!early0) fetch(t0, 0);
-    if (!(early0 && early1)) fetch(t0 + stride, 1);
+    for (uint32_t u = ahead; u < stages; u++) fetch(t0 + u * stride, u);
     __syncthreads();
     if (APPEND && blockIdx.x == 0 && h0 == g * rep && pos < a.positions) {
         uint16_t *dk = (uint16_t*)a.state + (size_t)(pos % a.ring) * row + g * a.dim;
@@ -241,8 +338,8 @@ window_step_kernel(const WindowArgs a) {
     const float sc = a.scale * 1.44269504088896340736f;           // scores in powers of two
     const uint32_t qaddr = smem_addr(sq + (lane & 15) * rk + (lane >> 4) * 8);
     uint32_t stage = 0;
-    for (uint32_t t = t0; t < t_end; t += stride, stage ^= 1) {
-        if (VEC) cp_wait<1>();
+    for (uint32_t t = t0; t < t_end; t += stride) {
+        if (VEC) { if (stages == 2) cp_wait<1>(); else if (stages == 3) cp_wait<2>(); else cp_wait<3>(); }
         uint16_t *k = my + stage * tile_el, *v = k + SP * rk;
         if (APPEND && t + 1 == t_end) {                           // this row's own key and value
             const uint32_t p = pos % SP;
@@ -251,15 +348,21 @@ window_step_kernel(const WindowArgs a) {
             for (uint32_t i = lane; i < a.vdim; i += 32) v[p * rv + i] = snew[dp + i];
         }
         __syncwarp();
-        float s[2][4] = {};
+        float s[2][4] = {}, s2[2][4] = {};                        // even and odd k steps: two chains of products
         const uint32_t kaddr = smem_addr(k + ((lane & 7) + (lane >> 4) * 8) * rk + ((lane >> 3) & 1) * 8);
 #pragma unroll 4
-        for (uint32_t ks = 0; ks < dp / 16; ks++) {
+        for (uint32_t ks = 0; ks < dp / 16; ks += 2) {
             uint32_t qa[4], b[4];
             ldsm4(qa, qaddr + ks * 32);
             ldsm4(b, kaddr + ks * 32);
             mma_bf16(s[0], qa, b[0], b[1]);
             mma_bf16(s[1], qa, b[2], b[3]);
+            if (ks + 1 < dp / 16) {
+                ldsm4(qa, qaddr + ks * 32 + 32);
+                ldsm4(b, kaddr + ks * 32 + 32);
+                mma_bf16(s2[0], qa, b[0], b[1]);
+                mma_bf16(s2[1], qa, b[2], b[3]);
+            }
         }
         float mx[2] = {m[0], m[1]};
 #pragma unroll
@@ -267,7 +370,7 @@ window_step_kernel(const WindowArgs a) {
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const uint32_t j = t * SP + i * 8 + 2 * t4 + (e & 1);
-                const float x = j >= first && j <= pos ? s[i][e] * sc : -INFINITY;
+                const float x = j >= first && j <= pos ? (s[i][e] + s2[i][e]) * sc : -INFINITY;
                 s[i][e] = x;
                 mx[e >> 1] = fmaxf(mx[e >> 1], x);
             }
@@ -301,106 +404,133 @@ window_step_kernel(const WindowArgs a) {
             uint32_t b[4];
             ldsm4_t(b, vaddr + i * 16);
             mma_bf16(o[i], ph, b[0], b[1]);
-            mma_bf16(o[i], pl, b[0], b[1]);
             mma_bf16(o[i + 1], ph, b[2], b[3]);
+            mma_bf16(o[i], pl, b[0], b[1]);
             mma_bf16(o[i + 1], pl, b[2], b[3]);
         }
         __syncwarp();
-        fetch(t + 2 * stride, stage);
+        fetch(t + stages * stride, stage);
+        stage = stage + 1 == stages ? 0 : stage + 1;
     }
     if (VEC) cp_wait<0>();
     __syncthreads();
-    // the warps' partial results: maximum, sum, values
+    // the warps' partial results: maximum, sum, values of the group's heads
 #pragma unroll
     for (int q = 0; q < 2; q++) {
         l[q] += __shfl_xor_sync(0xffffffffu, l[q], 1);
         l[q] += __shfl_xor_sync(0xffffffffu, l[q], 2);
-        if (t4 == 0) { wm[warp][g4 + 8 * q] = m[q]; wl[warp][g4 + 8 * q] = l[q]; }
-        float* d = acc + ((size_t)warp * 16 + g4 + 8 * q) * vp + 2 * t4;
+        const uint32_t h = g4 + 8 * q;
+        if (t4 == 0) { wm[warp][h] = m[q]; wl[warp][h] = l[q]; }
+        if (h >= nh) continue;
+        float* d = acc + ((size_t)warp * 16 + h) * vp + 2 * t4;
 #pragma unroll
         for (int i = 0; i < VT; i++) if (i * 8 < (int)vp) *(float2*)(d + i * 8) = make_float2(o[i][2 * q], o[i][2 * q + 1]);
     }
-    __syncthreads();
-    if (tid < 16) {
-        float mx = -INFINITY, sum = 0.0f;
-        for (uint32_t w = 0; w < SW; w++) mx = fmaxf(mx, wm[w][tid]);
-        for (uint32_t w = 0; w < SW; w++) {
-            const float f = wl[w][tid] > 0.0f ? exp2f(wm[w][tid] - mx) : 0.0f;      // a warp without tiles has sum 0
-            sum = fmaf(f, wl[w][tid], sum);
-            wm[w][tid] = f;
-        }
-        cm[tid] = mx; cl[tid] = sum;
-    }
+    // this CTA's share of the output, and its gates
+    const uint32_t per = (nh * a.vdim + C - 1) / C, e0 = blockIdx.x * per, e1 = min(e0 + per, nh * a.vdim);
+    const uint16_t* yg = a.gate_col == 0xFFFFFFFFu ? nullptr : (const uint16_t*)a.y + (size_t)r * a.y_cols + a.gate_col + h0 * a.vdim;
+    const float gate0 = yg && e0 + tid < e1 ? bf2f(__ldcg(yg + e0 + tid)) : 0.0f;
     __syncthreads();
     for (uint32_t i = tid; i < nh * vp; i += 256) {
         const uint32_t h = i / vp;
-        float s = 0.0f;
+        float f[SW], mx = -INFINITY, sum = 0.0f, s = 0.0f;
 #pragma unroll
-        for (uint32_t w = 0; w < SW; w++) s = fmaf(wm[w][h], acc[(size_t)w * 16 * vp + i], s);
+        for (uint32_t w = 0; w < SW; w++) { f[w] = wm[w][h]; mx = fmaxf(mx, f[w]); }
+#pragma unroll
+        for (uint32_t w = 0; w < SW; w++) {
+            f[w] = f[w] > -INFINITY ? exp2f(f[w] - mx) : 0.0f;    // a warp without tiles has sum 0
+            sum = fmaf(f[w], wl[w][h], sum);
+            s = fmaf(f[w], acc[(size_t)w * 16 * vp + i], s);
+        }
         acc[i] = s;                                               // only this thread reads element i of any warp
+        if (i % vp == 0) { cm[h] = mx; cl[h] = sum; }
     }
     if (C > 1) cluster.sync(); else __syncthreads();
-    const uint16_t* yg = a.gate_col == 0xFFFFFFFFu ? nullptr : (const uint16_t*)a.y + (size_t)r * a.y_cols + a.gate_col + h0 * a.vdim;
     uint16_t* out = (uint16_t*)a.out + ((size_t)r * a.heads + h0) * a.vdim;
-    for (uint32_t i = blockIdx.x * 256 + tid; i < nh * a.vdim; i += C * 256) {
+    for (uint32_t i = e0 + tid; i < e1; i += 256) {
         const uint32_t h = i / a.vdim, c = i % a.vdim;
-        float pm[8], pl[8], pv[8], mx = -INFINITY, num = 0.0f, den = 0.0f;
+        float pm[MAXC], pl[MAXC], pv[MAXC], mx = -INFINITY, num = 0.0f, den = 0.0f;
 #pragma unroll
-        for (uint32_t k = 0; k < 8; k++) {
-            if (k >= C) break;
-            pm[k] = *cluster.map_shared_rank(cm + h, k);
-            pl[k] = *cluster.map_shared_rank(cl + h, k);
-            pv[k] = *cluster.map_shared_rank(acc + h * vp + c, k);
-            mx = fmaxf(mx, pm[k]);
+        for (uint32_t k = 0; k < MAXC; k++) {
+            const uint32_t from = k < C ? k : 0;
+            pm[k] = *cluster.map_shared_rank(cm + h, from);
+            pl[k] = *cluster.map_shared_rank(cl + h, from);
+            pv[k] = *cluster.map_shared_rank(acc + h * vp + c, from);
         }
 #pragma unroll
-        for (uint32_t k = 0; k < 8; k++) {
-            if (k >= C) break;
-            const float f = pl[k] > 0.0f ? exp2f(pm[k] - mx) : 0.0f;
+        for (uint32_t k = 0; k < MAXC; k++) mx = fmaxf(mx, pm[k]);
+#pragma unroll
+        for (uint32_t k = 0; k < MAXC; k++) {
+            const float f = k < C && pl[k] > 0.0f ? exp2f(pm[k] - mx) : 0.0f;
             num = fmaf(f, pv[k], num);
             den = fmaf(f, pl[k], den);
         }
-        out[i] = f2bf(num / den * (yg ? sigmoid_f(bf2f(__ldcg(yg + i))) : 1.0f));
+        const float gt = !yg ? 1.0f : sigmoid_fast(i == e0 + tid ? gate0 : bf2f(__ldcg(yg + i)));
+        out[i] = f2bf(num / den * gt);
     }
     if (C > 1) cluster.sync();                                    // nobody leaves while its results are being read
 }
 
-size_t step_smem(const WindowArgs& a) {
+size_t step_smem(const WindowArgs& a, uint32_t stages, bool lp) {
     const size_t dp = (a.dim + 15u) & ~15u, vp = (a.vdim + 15u) & ~15u, rk = dp + 8, rv = vp + 8;
-    return (16 * rk + dp + vp) * 2 + SW * (((a.dim + 2) + 3u) & ~3u) * 4 + SW * 2 * SP * (rk + rv) * 2;
+    return (16 * rk + dp + vp) * 2 + (lp ? 0 : SW * (((a.dim + 2) + 3u) & ~3u) * 4) + SW * stages * SP * (rk + rv) * 2;
 }
 
 bool vec_rows(const WindowArgs& a) { return a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ring % SP == 0; }
 
-template <int VT, bool VEC, bool APPEND>
+constexpr size_t kStepSmem = 224 * 1024;
+
+template <int VT, bool VEC, bool APPEND, int LP>
 bool launch_step(cudaStream_t st, const WindowArgs& a, uint32_t rows) {
-    static int have[64] = {};
-    const size_t smem = step_smem(a);
-    if (!ensure_dyn_smem(window_step_kernel<VT, VEC, APPEND>, smem, have)) return false;
-    // two tiles per warp before another CTA helps
-    const uint32_t tiles = (a.window < a.ring ? a.window : a.ring) / SP + 1;
-    uint32_t C = 1;
+    static int have[64] = {}, wide[64] = {};       // wide: clusters of 16 CTAs the device can hold at once, + 1
+    const uint32_t tiles = (a.window < a.ring ? a.window : a.ring) / SP + 1, rep = a.heads / a.kv_heads;
+    const uint32_t clusters = a.kv_heads * ((rep + 15) / 16) * rows;
+    // two tiles per warp before another CTA helps, as many stages as fit (and as a warp has tiles)
+    uint32_t C = 1, stages = 4;
     while (C < 8 && C * SW * 2 < tiles) C *= 2;
-    const uint32_t rep = a.heads / a.kv_heads;
+    while (stages > 2 && step_smem(a, stages, LP) > kStepSmem) stages--;
+    const size_t smem = step_smem(a, stages, LP);
+    auto kernel = window_step_kernel<VT, VEC, APPEND, LP>;
+    if (!ensure_dyn_smem(kernel, smem, have)) return false;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(C, a.kv_heads * ((rep + 15) / 16), rows); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
-    if (launch_pdl_cluster(window_step_kernel<VT, VEC, APPEND>, cfg, dim3(C, 1, 1), a) != cudaSuccess) { cudaGetLastError(); return false; }
+    cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    int dev = 0;
+    if (C == 8 && tiles >= 16 * SW * 2 && cudaGetDevice(&dev) == cudaSuccess && dev >= 0 && dev < 64) {
+        if (!wide[dev]) {
+            int n = 0;
+            cudaLaunchAttribute at;
+            at.id = cudaLaunchAttributeClusterDimension;
+            at.val.clusterDim.x = 16; at.val.clusterDim.y = 1; at.val.clusterDim.z = 1;
+            cudaLaunchConfig_t q = cfg;
+            q.gridDim = dim3(16); q.attrs = &at; q.numAttrs = 1;
+            if (cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess ||
+                cudaOccupancyMaxActiveClusters(&n, kernel, &q) != cudaSuccess) { cudaGetLastError(); n = 0; }
+            wide[dev] = n + 1;
+        }
+        if ((uint32_t)(wide[dev] - 1) >= clusters) C = 16;
+    }
+    cfg.gridDim = dim3(C, a.kv_heads * ((rep + 15) / 16), rows);
+    if (launch_pdl_cluster(kernel, cfg, dim3(C, 1, 1), a, stages) != cudaSuccess) { cudaGetLastError(); return false; }
     g_launches++;
     return true;
 }
 
 template <bool APPEND>
 bool step(cudaStream_t st, const WindowArgs& a, uint32_t rows) {
-    if (!a.bf16 || a.vdim > 256 || step_smem(a) > 220 * 1024) return false;
+    if (!a.bf16 || a.vdim > 256 || step_smem(a, 2, false) > kStepSmem) return false;
     const uint32_t vt = (a.vdim + 15) / 16 * 2;
     if (vec_rows(a)) {
-        if (vt <= 8) return launch_step<8, true, APPEND>(st, a, rows);
-        if (vt <= 16) return launch_step<16, true, APPEND>(st, a, rows);
-        return launch_step<32, true, APPEND>(st, a, rows);
+        if (APPEND && head_vec(a) && vt <= 16) {
+            if (a.dim == 64) return vt <= 8 ? launch_step<8, true, APPEND, 8>(st, a, rows) : launch_step<16, true, APPEND, 8>(st, a, rows);
+            if (a.dim == 128) return vt <= 8 ? launch_step<8, true, APPEND, 16>(st, a, rows) : launch_step<16, true, APPEND, 16>(st, a, rows);
+        }
+        if (vt <= 8) return launch_step<8, true, APPEND, 0>(st, a, rows);
+        if (vt <= 16) return launch_step<16, true, APPEND, 0>(st, a, rows);
+        return launch_step<32, true, APPEND, 0>(st, a, rows);
     }
-    if (vt <= 8) return launch_step<8, false, APPEND>(st, a, rows);
-    if (vt <= 16) return launch_step<16, false, APPEND>(st, a, rows);
-    return launch_step<32, false, APPEND>(st, a, rows);
+    if (vt <= 8) return launch_step<8, false, APPEND, 0>(st, a, rows);
+    if (vt <= 16) return launch_step<16, false, APPEND, 0>(st, a, rows);
+    return launch_step<32, false, APPEND, 0>(st, a, rows);
 }
 
 }  // namespace
@@ -410,14 +540,24 @@ bool k_window_flash(cudaStream_t st, const WindowArgs& a, uint32_t rows);
 
 void k_heads_append(cudaStream_t st, const WindowArgs& a, uint32_t rows) {
     if (!rows) return;
+    const uint32_t lp = a.dim / 8;
+    if (head_vec(a)) {
+        const dim3 grid(rows, ((a.heads + a.kv_heads) * lp + a.kv_heads * (a.vdim / 8) + 255) / 256);
+        if (lp == 8) launch_pdl(heads_append_vec_kernel<8>, grid, dim3(256), 0, st, a);
+        else if (lp == 16) launch_pdl(heads_append_vec_kernel<16>, grid, dim3(256), 0, st, a);
+        else launch_pdl(heads_append_vec_kernel<32>, grid, dim3(256), 0, st, a);
+        g_launches++;
+        return;
+    }
     const size_t smem = 8 * (size_t)(a.dim + 1) * 4;
+    const dim3 grid(rows, (a.heads + 2 * a.kv_heads + 7) / 8);
     static int have_b[64] = {}, have_f[64] = {};
     if (a.bf16) {
         if (smem > 40 * 1024) ensure_dyn_smem(heads_append_kernel<ActBf16>, smem, have_b);
-        launch_pdl(heads_append_kernel<ActBf16>, dim3(rows), dim3(256), smem, st, a);
+        launch_pdl(heads_append_kernel<ActBf16>, grid, dim3(256), smem, st, a);
     } else {
         if (smem > 40 * 1024) ensure_dyn_smem(heads_append_kernel<ActF32>, smem, have_f);
-        launch_pdl(heads_append_kernel<ActF32>, dim3(rows), dim3(256), smem, st, a);
+        launch_pdl(heads_append_kernel<ActF32>, grid, dim3(256), smem, st, a);
     }
     g_launches++;
 }
@@ -426,7 +566,7 @@ void k_window_attend(cudaStream_t st, const WindowArgs& a, uint32_t rows, bool e
     if (!rows) return;
     if (a.bf16 && !exact) {
         if (rows <= kStepRows && step<false>(st, a, rows)) return;
-        if (k_window_flash(st, a, rows)) return;
+        if (k_window_sm100(st, a, rows) || k_window_flash(st, a, rows)) return;
     }
     const size_t smem = (size_t)(a.dim + a.vdim) * 4;
     static int have_b[64] = {}, have_f[64] = {};

@@ -161,9 +161,9 @@ window_flash_kernel(const WindowArgs a, uint32_t rows) {
         for (int i = 0; i < VT; i++) {
             const uint32_t c = i * 8 + 2 * t4;
             if (c >= a.vdim) break;
-            const float u = o[i][2 * r] * f * (gate ? sigmoid_f(bf2f(__ldcg(yg + c))) : 1.0f);
+            const float u = o[i][2 * r] * f * (gate ? sigmoid_fast(bf2f(__ldcg(yg + c))) : 1.0f);
             if (c + 1 >= a.vdim) { out[c] = f2bf(u); break; }
-            const float w = o[i][2 * r + 1] * f * (gate ? sigmoid_f(bf2f(__ldcg(yg + c + 1))) : 1.0f);
+            const float w = o[i][2 * r + 1] * f * (gate ? sigmoid_fast(bf2f(__ldcg(yg + c + 1))) : 1.0f);
             if (VEC) *(uint32_t*)(out + c) = pack_bf2(u, w);
             else { out[c] = f2bf(u); out[c + 1] = f2bf(w); }
         }
