@@ -1090,25 +1090,26 @@ def run_design(args, width):
     ms = timed(step)
     add(cfg.name, "prefill 2048", ms, S_, units(eng, ids, man["hidden_temp"], work_fixed(S_, S_)))
     eng.shutdown()
-    buf, man = build_decode_runlist(cfg, 1, CTX, quant="f16")
-    eng = Engine(lib, buf)
-    for li in range(4):
-        kv = torch.randn(CTX * 2 * 1024, device="cuda", dtype=torch.float16)
-        assert lib.gehtp_cuda_state_load(ctypes.byref(eng.blob), li, kv.data_ptr(), kv.numel() * 2, 1, 1024, CTX - 64, err, 256) == 0, err.value
-    face = decode_face(man, [7], CTX - 64, 128, 1e6)
-    dface = torch.from_numpy(face.view(np.int16).copy()).cuda()
-    out = torch.zeros(4, dtype=torch.int16, device="cuda")
-
-    def rewind():
+    for C in (CTX,) if args.design == "Ripidra" else (CTX, 1088):      # 1088: beside windows of 1024
+        buf, man = build_decode_runlist(cfg, 1, C, quant="f16")
+        eng = Engine(lib, buf)
         for li in range(4):
-            assert lib.gehtp_cuda_state_set_count(li, CTX - 64) == 0
+            kv = torch.randn(C * 2 * 1024, device="cuda", dtype=torch.float16)
+            assert lib.gehtp_cuda_state_load(ctypes.byref(eng.blob), li, kv.data_ptr(), kv.numel() * 2, 1, 1024, C - 64, err, 256) == 0, err.value
+        face = decode_face(man, [7], C - 64, 128, 1e6)
+        dface = torch.from_numpy(face.view(np.int16).copy()).cuda()
+        out = torch.zeros(4, dtype=torch.int16, device="cuda")
 
-    def step():
-        assert lib.gehtp_cuda_run_dev(ctypes.byref(eng.blob), dface.data_ptr(), out.data_ptr(), man["token_temp"], err, 256) == 0, err.value
-    ms = timed(step, rewind)
-    rewind()
-    add(cfg.name, "decode ctx %d" % (CTX - 64), ms, 1, units(eng, face, man["token_temp"], work_fixed(1, CTX)))
-    eng.shutdown()
+        def rewind():
+            for li in range(4):
+                assert lib.gehtp_cuda_state_set_count(li, C - 64) == 0
+
+        def step():
+            assert lib.gehtp_cuda_run_dev(ctypes.byref(eng.blob), dface.data_ptr(), out.data_ptr(), man["token_temp"], err, 256) == 0, err.value
+        ms = timed(step, rewind)
+        rewind()
+        add(cfg.name, "decode ctx %d" % (C - 64), ms, 1, units(eng, face, man["token_temp"], work_fixed(1, C - 64)))
+        eng.shutdown()
     if args.design != "Ripidra":
         return lines
     # ---- the delta rule of the gated-delta layer (config 5) at the same heads: chunks of 64 tokens, convolution over 3 H 128 channels

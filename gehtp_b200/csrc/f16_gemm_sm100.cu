@@ -311,6 +311,16 @@ bool launch(cudaStream_t st, const uint16_t* a, uint32_t lda, const uint16_t* w,
             if (cost < best) { best = cost; S = c; }
         }
     }
+    // sums that go through memory anyway: also where the tiles fill the SMs but their last round would not
+    if (Heavy<E>::value && tiles >= (uint32_t)sms) {
+        const float run_cost = (float)((double)M * np * sizeof(float) / 2e6);      // one more run to write and read, in k blocks
+        float best = (float)((tiles + sms - 1) / sms) * (float)(KG + 4);
+        for (uint32_t c = 2; c <= 4; c++) {
+            if (KG % c || KG / c < (uint32_t)C::STAGES || (size_t)c * M * np * sizeof(float) > ((size_t)64 << 20)) continue;
+            const float cost = (float)((tiles * c + sms - 1) / sms) * (float)(KG / c + 4) + (float)(c - 1) * run_cost;
+            if (cost < best) { best = cost; S = c; }
+        }
+    }
     float* part = nullptr;
     if (S > 1 || Heavy<E>::value) {
         SplitScratch* ss = split_scratch(st, (size_t)S * M * np * sizeof(float));
